@@ -25,14 +25,19 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "--use_fast_math", "-Xptxas", "-v",
 ]
 # --use_fast_math is dropped for files whose numerics are compared bit-for-bit with an oracle
-NO_FAST_MATH = {"act_quant.cu"}
+# (act_quant) or that also carry the 32-bit form of a model
+NO_FAST_MATH = {"act_quant.cu", "bf16_gemm.cu", "bf16_gemm_decode.cu", "f32_gemm.cu", "rotary_paged.cu", "attn_paged.cu"}
 GXX_FLAGS = ["-O2", "-std=c++20", "-fPIC", "-Wall", "-Wextra", "-fno-stack-protector", "-pthread"]
 
 KERNEL_LIB = "libb200_kernels.so"
 # Variants of the kernel library: same sources, one extra define each.  "trace": in-kernel %globaltimer stamps
 # (csrc/kernels/trace.cuh); "debug": range checks on peer / scratch accesses that record the bad offset in the status
 # word and skip the access (csrc/kernels/debug_check.h).  The production library has neither.
-KERNEL_VARIANTS = {"": [], "trace": ["-DB200RT_TRACE"], "debug": ["-DB200RT_DEBUG"]}
+# "dense": production flags, but only the kernels of the unquantised (bf16 / fp32) models: what a tool that serves one
+# such model from a fresh checkout compiles.
+KERNEL_VARIANTS = {"": [], "trace": ["-DB200RT_TRACE"], "debug": ["-DB200RT_DEBUG"], "dense": []}
+KERNEL_SUBSETS = {"dense": ("attn_decode_paged.cu", "attn_paged.cu", "attn_prefill_paged.cu", "bf16_gemm.cu", "bf16_gemm_decode.cu",
+                            "f32_gemm.cu", "rope_kv.cu", "rotary_paged.cu", "tmap.cu", "trace.cu")}
 
 
 HOSTRT_LIB = "libb200_hostrt.so"
@@ -80,10 +85,10 @@ def _stale(stamp: Path, digest: str, product: Path) -> bool:
 def build_kernels(verbose: bool = False, variant: str = "") -> Path:
     """Compile every .cu under csrc/kernels for sm_100a and link libb200_kernels[_variant].so."""
     srcdir = CSRC / "kernels"
-    sources = sorted(srcdir.glob("*.cu"))
+    sources = [s for s in sorted(srcdir.glob("*.cu")) if s.name in KERNEL_SUBSETS.get(variant, (s.name,))]
     headers = sorted(list(srcdir.glob("*.cuh")) + list(srcdir.glob("*.h")) + list((CSRC / "fabric").glob("*.h")))
     LIBDIR.mkdir(parents=True, exist_ok=True)
-    objdir = OBJDIR / variant if variant else OBJDIR
+    objdir = OBJDIR / variant if KERNEL_VARIANTS[variant] else OBJDIR       # a subset shares the production objects
     objdir.mkdir(parents=True, exist_ok=True)
     nvcc = _nvcc()
     vflags = NVCC_FLAGS + KERNEL_VARIANTS[variant]
@@ -106,11 +111,20 @@ def build_kernels(verbose: bool = False, variant: str = "") -> Path:
         objs = list(ex.map(compile_one, sources))
     lib = LIBDIR / kernel_lib_name(variant)
     link_digest = _digest(objs, "link")
-    stamp = objdir / "kernels.link.stamp"
+    stamp = objdir / (lib.stem + ".link.stamp")
     if _stale(stamp, link_digest, lib):
         _run([nvcc, "-shared", "-o", str(lib), *map(str, objs), "-cudart", "static"])
         stamp.write_text(json.dumps({"digest": link_digest}))
     return lib
+
+
+def ensure_kernels(variant: str) -> Path:
+    """Build the kernel library if its sources changed; concurrent callers wait for each other."""
+    import fcntl
+    OBJDIR.mkdir(parents=True, exist_ok=True)
+    with open(OBJDIR / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build_kernels(variant=variant)
 
 
 def _build_cpp(name: str, subdir: str, extra_flags=(), libs=()) -> Path:

@@ -100,6 +100,8 @@ int b200_rope_kv_write(const void* qkv, long long ld_qkv, const int* positions, 
 int b200_embed_gather(const long long* ids, const void* table, void* out, int M, int d, int vocab, cudaStream_t stream);
 int b200_argmax_rows(const void* logits, long long ld, int rows, int n, int index_offset, int chunks, float* out_val,
                      long long* out_idx, cudaStream_t stream);
+int b200_argmax_rows_f32(const float* logits, long long ld, int rows, int n, int index_offset, int chunks, float* out_val,
+                         long long* out_idx, cudaStream_t stream);
 int b200_argmax_merge(const float* cand_val, const long long* cand_idx, int world, int rows, long long* out_idx,
                       cudaStream_t stream);
 size_t b200_attn_decode_scratch_floats(int B, int hq, int splits);
@@ -220,6 +222,62 @@ int b200_ep_combine_reduce(const int* ids_local, int M, int k, int d, int expert
                            void* const* peer_data, int world, int rank, size_t recv_off0, size_t recv_off1,
                            size_t ctr_off, int r_cap, void* words, void* out, long long ldo, int* status,
                            int limit_ms, int num_sms, cudaStream_t stream);
+
+// ---- dense (unquantised) linears with a fused epilogue, dense_epilogue.cuh ---------------------------------------------
+enum { B200_EPI_STORE = 0, B200_EPI_RESIDUAL = 1, B200_EPI_GLU = 2 };
+typedef struct b200_dense_epilogue {
+  int mode;
+  int out_f32;                          // element type of y: 0 bf16, 1 fp32
+  int exact;                            // library tanh / exp instead of the approximate hardware functions
+  void* y; long long ldy;               // store: result; glu: [M][N/2]; residual: normalised rows, or NULL
+  float* x; long long ldx;              // residual: the fp32 stream, updated in place
+  const float* add;                     // residual: second addend with the pitch of x, or NULL
+  float mult;                           // residual: factor on the linear's result
+  const float* norm_w; const float* norm_b; float norm_alpha;     // dynamic tanh: tanh(alpha x) w + b
+  float limit;                          // glu: bound of both branches
+} b200_dense_epilogue;
+// x [M][K] and w [N][K] with row pitches in elements (multiples of 8 for bf16, 16-byte aligned); force_bn 0 or 64 / 128 / 256.
+int b200_bf16_gemm(const void* x, long long ldx, const void* w, long long ldw, int M, int N, int K,
+                   const b200_dense_epilogue* epi, int* status, int num_sms, int force_bn, cudaStream_t stream);
+int b200_bf16_gemm_decode(const void* x, long long ldx, const void* w, long long ldw, int M, int N, int K,
+                          const b200_dense_epilogue* epi, int* status, int num_sms, int splits, cudaStream_t stream);
+int b200_f32_gemm(const float* x, long long ldx, const float* w, long long ldw, int M, int N, int K,
+                  const b200_dense_epilogue* epi, cudaStream_t stream);
+
+// ---- attention over a paged cache with free head sizes, optional chunk mask, sink and output gate ------------------------
+typedef struct b200_paged_cache {
+  void* data; int f32;                  // records of kv_heads * page_size * (dk + dv) elements (bf16 or fp32)
+  int kv_heads, page_size, dk, dv;      // dk, dv multiples of 8
+  int num_pages;
+  const int* page_table; int num_seqs, max_pages;      // [num_seqs][max_pages]
+} b200_paged_cache;
+typedef struct b200_attn_spec {
+  float scale;
+  int chunk;                            // > 0: a position sees only its own block of `chunk` positions; 0: all earlier ones
+  const float* sink;                    // [hq] extra exponent in the denominator, or NULL
+  const void* gate; long long ldg;      // [M][hq] gate logits (element type of q): head outputs times sigmoid, or NULL
+} b200_attn_spec;
+int b200_rotary_paged(void* qkv, long long ld, int hq, int M, const int* positions, const int* seq_ids,
+                      const float* cos_tab, const float* sin_tab, int pairs, int interleaved, int max_pos,
+                      const b200_paged_cache* cache, int* status, cudaStream_t stream);
+int b200_embed_norm(const long long* ids, const void* table, long long ldt, int vocab, int table_f32, float scale,
+                    int M, int d, float* x, float* copy, const b200_dense_epilogue* norm, cudaStream_t stream);
+// General form (any head size up to 512, bf16 or fp32): one warp per (token, head).  q [M][hq][dk] with row pitch ldq;
+// out [M][hq][dv] with row pitch ldo.  seq_ids NULL: token i belongs to sequence i; positions < 0 are skipped.
+int b200_attn_paged(const void* q, long long ldq, void* out, long long ldo, int hq, int M, const int* positions,
+                    const int* seq_ids, const int* seq_lens, const b200_paged_cache* cache, const b200_attn_spec* spec,
+                    int* status, cudaStream_t stream);
+// Prefill portions on the tensor cores (bf16, dk and dv up to 128, page size 16): rows [cu[b], cu[b+1]) are consecutive
+// positions of one sequence whose keys up to there are in the cache already.
+int b200_attn_prefill_paged(const void* q, long long ldq, void* out, long long ldo, int hq, int M, int B, int max_len,
+                            const int* cu_seqlens, const int* positions, const int* seq_ids,
+                            const b200_paged_cache* cache, const b200_attn_spec* spec, int* status, cudaStream_t stream);
+// One new token per sequence (row b of qkv = sequence b; bf16, dk and dv up to 256, page size 16): rotary embedding, cache
+// append, attention, sink and gate in one launch.  seq_lens[b] counts the new token; 0: empty slot, zero output.
+int b200_attn_decode_paged(const void* qkv, long long ld, void* out, long long ldo, int hq, int B, const int* positions,
+                           const int* seq_lens, const float* cos_tab, const float* sin_tab, int pairs, int interleaved,
+                           int max_pos, const b200_paged_cache* cache, const b200_attn_spec* spec, int splits,
+                           int* status, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

@@ -1,0 +1,85 @@
+// What happens to a finished value of a dense (unquantised) linear before it leaves the kernel.
+//
+//   store     y[m][n] = v
+//   residual  x[m][n] += mult * v (fp32, in place), optionally + add[m][n]; then, if y is given, the norm of the *next*
+//             sub-layer is applied to the new residual and y[m][n] = norm(x) - possible here because the norm is
+//             element-wise (dynamic tanh), so no second pass over the row is needed
+//   glu       columns 2c / 2c+1 are gate / up of channel c (weight rows interleaved at load time):
+//             y[m][c] = g sigmoid(1.702 g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit)
+//
+// Every buffer has a row pitch of at least N rounded up to four elements and 16-byte aligned rows, so a group of four
+// columns is always handled as one vector; columns beyond N land in the padding.
+#pragma once
+#include <cuda_runtime.h>
+#include <cuda_bf16.h>
+#include <stdint.h>
+#include "api.h"
+
+namespace b200 {
+
+__device__ __forceinline__ float epi_sigmoid(float z, bool exact) {
+  return exact ? 1.f / (1.f + expf(-z)) : __fdividef(1.f, 1.f + __expf(-z));
+}
+// tanh(z) = 1 - 2 / (e^2z + 1): absolute error of a few 1e-7, far below the bf16 rounding that follows; the 32-bit build
+// of the model takes the library function.  z is bounded so that e^2z stays inside what __fdividef accepts.
+__device__ __forceinline__ float epi_tanh(float z, bool exact) {
+  if (exact) return tanhf(z);
+  z = fminf(fmaxf(z, -15.f), 15.f);
+  return 1.f - __fdividef(2.f, __expf(2.f * z) + 1.f);
+}
+
+__device__ __forceinline__ void store4_any(void* base, bool f32, long long off, float4 v) {
+  if (f32) {
+    *reinterpret_cast<float4*>(static_cast<float*>(base) + off) = v;
+  } else {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 raw;
+    raw.x = *reinterpret_cast<uint32_t*>(&lo);
+    raw.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(base) + off) = raw;
+  }
+}
+
+// element-wise norm of four residual values of columns n .. n+3
+__device__ __forceinline__ float4 epi_norm4(const b200_dense_epilogue& e, int n, float4 x, bool exact) {
+  const float4 w = __ldg(reinterpret_cast<const float4*>(e.norm_w + n));
+  const float4 b = __ldg(reinterpret_cast<const float4*>(e.norm_b + n));
+  float4 o;
+  o.x = epi_tanh(e.norm_alpha * x.x, exact) * w.x + b.x;
+  o.y = epi_tanh(e.norm_alpha * x.y, exact) * w.y + b.y;
+  o.z = epi_tanh(e.norm_alpha * x.z, exact) * w.z + b.z;
+  o.w = epi_tanh(e.norm_alpha * x.w, exact) * w.w + b.w;
+  return o;
+}
+
+// columns n .. n+3 (n a multiple of four, n < N) of row m
+__device__ __forceinline__ void epi_apply4(const b200_dense_epilogue& e, long long m, int n, float4 v) {
+  const bool f32 = e.out_f32 != 0;
+  if (e.mode == B200_EPI_STORE) {
+    store4_any(e.y, f32, m * e.ldy + n, v);
+  } else if (e.mode == B200_EPI_GLU) {
+    const bool exact = e.exact != 0;
+    const float g0 = fminf(v.x, e.limit), u0 = fminf(fmaxf(v.y, -e.limit), e.limit);
+    const float g1 = fminf(v.z, e.limit), u1 = fminf(fmaxf(v.w, -e.limit), e.limit);
+    const float o0 = g0 * epi_sigmoid(1.702f * g0, exact) * (u0 + 1.f);
+    const float o1 = g1 * epi_sigmoid(1.702f * g1, exact) * (u1 + 1.f);
+    const long long off = m * e.ldy + (n >> 1);
+    if (f32) {
+      *reinterpret_cast<float2*>(static_cast<float*>(e.y) + off) = make_float2(o0, o1);
+    } else {
+      *reinterpret_cast<__nv_bfloat162*>(static_cast<__nv_bfloat16*>(e.y) + off) = __floats2bfloat162_rn(o0, o1);
+    }
+  } else {
+    float4* xp = reinterpret_cast<float4*>(e.x + m * e.ldx + n);
+    float4 x = *xp;
+    x.x += e.mult * v.x; x.y += e.mult * v.y; x.z += e.mult * v.z; x.w += e.mult * v.w;
+    if (e.add) {
+      const float4 a = *reinterpret_cast<const float4*>(e.add + m * e.ldx + n);
+      x.x += a.x; x.y += a.y; x.z += a.z; x.w += a.w;
+    }
+    *xp = x;
+    if (e.y) store4_any(e.y, f32, m * e.ldy + n, epi_norm4(e, n, x, e.exact != 0));
+  }
+}
+
+}  // namespace b200

@@ -13,5 +13,8 @@ constexpr int SWAP_MAX_M = 64;  // up to this many tokens the weights fill the M
 
 // 2-D row-major byte matrix [rows][cols] with row pitch `pitch` bytes; box = 128 bytes x box_rows, 128-byte swizzle.
 int make_tmap_2d_u8(CUtensorMap* out, const void* base, uint64_t cols, uint64_t rows, uint64_t pitch, uint32_t box_rows);
+// bf16 [n2][n1][n0] with pitches in bytes; box = 64 columns x rows1 x rows2, 128-byte swizzle, zero fill outside.
+int make_tmap_3d_bf16(CUtensorMap* out, const void* base, uint64_t n0, uint64_t n1, uint64_t n2, uint64_t pitch1,
+                      uint64_t pitch2, uint32_t rows1, uint32_t rows2);
 
 }  // namespace b200

@@ -125,9 +125,12 @@ __global__ void embed_gather_kernel(const long long* ids, const __nv_bfloat16* t
 
 // grid (rows, chunks): CTA (r, c) scans columns [c*cs, (c+1)*cs) of row r and writes candidate [c][r];
 // ties resolve to the lowest index (matches torch.argmax on a single device after the merge)
-__global__ void __launch_bounds__(256) argmax_rows_kernel(const __nv_bfloat16* logits, long long ld, int n,
-                                                          int chunk, int index_offset, float* out_val,
-                                                          long long* out_idx) {
+__device__ __forceinline__ float logit_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float logit_f(float v) { return v; }
+
+template <typename T>
+__global__ void __launch_bounds__(256) argmax_rows_kernel(const T* logits, long long ld, int n, int chunk, int index_offset,
+                                                          float* out_val, long long* out_idx) {
   pdl_launch_dependents();   // the next kernel may start its prologue now
   pdl_wait();                // everything before this kernel in the stream has completed
 
@@ -135,11 +138,11 @@ __global__ void __launch_bounds__(256) argmax_rows_kernel(const __nv_bfloat16* l
   __shared__ int si[8];
   const int row = blockIdx.x;
   const int c0 = blockIdx.y * chunk, c1 = min(n, c0 + chunk);
-  const __nv_bfloat16* x = logits + static_cast<size_t>(row) * ld;
+  const T* x = logits + static_cast<size_t>(row) * ld;
   float best = -INFINITY;
   int bi = 0x7fffffff;
   auto consider = [&](float v, int i) { if (v > best || (v == best && i < bi)) { best = v; bi = i; } };
-  if (((reinterpret_cast<uintptr_t>(x) | static_cast<uintptr_t>(c0 * 2)) & 15) == 0) {
+  if (sizeof(T) == 2 && ((reinterpret_cast<uintptr_t>(x) | static_cast<uintptr_t>(c0 * 2)) & 15) == 0) {
     const int nv = (c1 - c0) / 8;
     const uint4* xv = reinterpret_cast<const uint4*>(x + c0);
     for (int i = threadIdx.x; i < nv; i += blockDim.x) {
@@ -151,9 +154,9 @@ __global__ void __launch_bounds__(256) argmax_rows_kernel(const __nv_bfloat16* l
         consider(__uint_as_float(w[k] & 0xffff0000u), c0 + i * 8 + 2 * k + 1);
       }
     }
-    for (int i = c0 + nv * 8 + threadIdx.x; i < c1; i += blockDim.x) consider(__bfloat162float(x[i]), i);
+    for (int i = c0 + nv * 8 + threadIdx.x; i < c1; i += blockDim.x) consider(logit_f(x[i]), i);
   } else {
-    for (int i = c0 + threadIdx.x; i < c1; i += blockDim.x) consider(__bfloat162float(x[i]), i);
+    for (int i = c0 + threadIdx.x; i < c1; i += blockDim.x) consider(logit_f(x[i]), i);
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
@@ -230,7 +233,18 @@ extern "C" int b200_argmax_rows(const void* logits, long long ld, int rows, int 
   if (rows <= 0) return 0;
   if (chunks < 1) chunks = 1;
   const int chunk = ((n + chunks - 1) / chunks + 7) & ~7;
-  launch_ex(argmax_rows_kernel, dim3(dim3(rows, chunks)), dim3(256), 0, stream, 0, static_cast<const __nv_bfloat16*>(logits), ld, n, chunk, index_offset, out_val, out_idx);
+  launch_ex(argmax_rows_kernel<__nv_bfloat16>, dim3(dim3(rows, chunks)), dim3(256), 0, stream, 0, static_cast<const __nv_bfloat16*>(logits), ld, n, chunk, index_offset, out_val, out_idx);
+  cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -2000 - static_cast<int>(e);
+}
+
+// the same over fp32 logits
+extern "C" int b200_argmax_rows_f32(const float* logits, long long ld, int rows, int n, int index_offset, int chunks,
+                                    float* out_val, long long* out_idx, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (chunks < 1) chunks = 1;
+  const int chunk = ((n + chunks - 1) / chunks + 7) & ~7;
+  launch_ex(argmax_rows_kernel<float>, dim3(dim3(rows, chunks)), dim3(256), 0, stream, 0, logits, ld, n, chunk, index_offset, out_val, out_idx);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -2000 - static_cast<int>(e);
 }

@@ -12,9 +12,9 @@ import os
 
 import torch
 
-from ..models.config import ModelConfig, RuntimeConfig
-from ..models.decoder import Decoder, KVState
-from ..models import weights as Wt
+from ..models.config import RuntimeConfig
+from ..models.kvcache import KVState
+from ..models.registry import family_of
 from ..ops.workspace import Workspace, default_workspace, has_default_workspace, install_default_workspace
 from ..parallel.comm import Comm
 from ..utils.trace import op_range
@@ -24,8 +24,10 @@ from .runtime import RankRuntime
 class Engine:
     _instances = 0
 
-    def __init__(self, cfg: ModelConfig, rt: RuntimeConfig | None = None, weights: dict | None = None, seed: int = 0,
+    def __init__(self, cfg, rt: RuntimeConfig | None = None, weights: dict | None = None, seed: int = 0,
                  device=None, comm: Comm | None = None):
+        """``cfg``: a configuration of any registered model family (``models.registry``)."""
+        family = family_of(cfg)
         self.cfg = cfg
         self.rt = rt or RuntimeConfig()
         self.comm = comm or Comm.single()
@@ -39,13 +41,13 @@ class Engine:
         self.runtime = RankRuntime(self.device)
         self.heartbeat = None
         if weights is None:
-            weights = Wt.random_shard(cfg, self.rt.tp, self.comm.rank, self.device, seed)
+            weights = family.random_weights(cfg, self.rt, self.comm.rank, self.device, seed)
         self.tp_ctx = None
         if self.comm.world > 1 and self.rt.fused_collectives:
             from ..parallel.tp import TPContext
             self.tp_ctx = TPContext(cfg.d_model, max_tokens=self.rt.max_prefill_tokens, group=self.comm.group,
                                     device=self.device, wait_limit_ms=self.rt.wait_limit_ms)
-        self.model = Decoder(cfg, self.rt, weights, self.comm, self.device, tp_ctx=self.tp_ctx)
+        self.model = family.model(cfg, self.rt, weights, self.comm, self.device, tp_ctx=self.tp_ctx)
         self.kv: KVState | None = None
         self.batch = 0
         self._graphs: dict[int, torch.cuda.CUDAGraph] = {}
@@ -57,6 +59,7 @@ class Engine:
         self._stream = torch.cuda.Stream(device=self.device)
         if self.comm.world > 1 and os.environ.get("B200RT_HEARTBEAT", "1") not in ("0", "false"):
             self._start_heartbeat()
+        self._graph_logits: dict[int, torch.Tensor | None] = {}      # what a captured decode step leaves in last_logits
         self._admitted = 0          # tokens per sequence the KV pages of the running batch can hold
         self._host_len = 0          # tokens per sequence already in the cache (host-side mirror of ``positions``)
 
@@ -70,6 +73,7 @@ class Engine:
         if self.kv is None or self.kv.seq_lens.numel() != batch or self.kv.max_pages * self.rt.page_size < max_total_len:
             self.kv = None                  # free the old cache before the new one is allocated
             self._graphs.clear()
+            self._graph_logits.clear()
             self._prefill_graphs.clear()
             self._place_buffers(batch)
             self.kv = KVState(self.cfg, self.rt, self.device, batch, self.rt.max_seq_len, alloc=self.runtime.zeros)
@@ -87,6 +91,7 @@ class Engine:
         self.kv.flush()
         self.batch = batch
         self._admitted = max_total_len
+        self._active_host = [0] * batch     # what ``active`` holds
         self._lens = [0] * batch            # tokens per slot already in the cache (host mirror of ``positions``); 0: empty
         self._host_len = 0                  # longest of them
 
@@ -133,18 +138,25 @@ class Engine:
             lens = [int(p.numel()) for p in prompts]
             if len(set(lens)) == 1:
                 prompts = torch.stack([p.reshape(-1) for p in prompts])
+            elif max(lens) > self.rt.max_prefill_tokens and self.model.supports_portions:
+                return self._prefill_portions(prompts)
             else:
                 return self._prefill_ragged(prompts, lens)
         B, S = prompts.shape
+        if S > self.rt.max_prefill_tokens and self.model.supports_portions:
+            return self._prefill_portions(list(prompts))
         if S + 1 > self._admitted:
             raise ValueError(f"a prompt of {S} tokens leaves no room to decode within the {self._admitted} admitted")
         for b in range(B):
+            if self._lens[b] > 0:
+                self._reset_slot(b)
             self.kv.admit(b, S + 1)
         self.kv.flush()
         self._prefill_equal(prompts.to(self.device, non_blocking=True), 0, use_graph)
         self.positions[:B].fill_(S)
         self.kv.seq_lens[:B].fill_(S + 1)      # the next decode step attends to the prompt plus its own token
         self.active[:B].fill_(1)
+        self._active_host[:B] = [1] * B
         for b in range(B):
             self._lens[b] = S
         self._host_len = max(self._lens)
@@ -190,6 +202,8 @@ class Engine:
         if max(lens) + 1 > self._admitted or min(lens) < 1:
             raise ValueError(f"prompt lengths {min(lens)}..{max(lens)} do not fit the {self._admitted} admitted tokens")
         for b in range(B):
+            if self._lens[b] > 0:
+                self._reset_slot(b)
             self.kv.admit(b, lens[b] + 1)
         self.kv.flush()
         dev = self.device
@@ -216,10 +230,120 @@ class Engine:
         self.positions[:B].copy_(lt)
         self.kv.seq_lens[:B].copy_(lt + 1)
         self.active[:B].fill_(1)
+        self._active_host[:B] = [1] * B
         for b in range(B):
             self._lens[b] = lens[b]
         self._host_len = max(self._lens)
         return self.tokens.clone()
+
+    def _prefill_portions(self, prompts) -> torch.Tensor:
+        """Prompts longer than one call may carry: every sequence from scratch, in portions."""
+        for b, p in enumerate(prompts):
+            if not 1 <= p.numel() < self._admitted:
+                raise ValueError(f"a prompt of {p.numel()} tokens does not fit the {self._admitted} admitted tokens")
+            self._reset_slot(b)
+            self._extend([(b, p.reshape(-1), [p.numel() - 1])])
+        return self.tokens[:len(prompts)].clone()
+
+    def _reset_slot(self, slot: int) -> None:
+        self.kv.release(slot)
+        self._lens[slot] = 0
+
+    # ---- explicit steps: given tokens in, logits out --------------------------------------------------------------
+    def step(self, entries, use_graph: bool = True) -> list[torch.Tensor]:
+        """Run given tokens: ``entries`` is a list of (slot, token ids, places); each slot's tokens continue what the slot
+        already holds (nothing, after ``start_batch`` or ``release_sequence``), and the fp32 logits at the ``places``
+        among them come back, one [len(places), vocab] tensor per entry.  Single tokens of running sequences go
+        through the decode step (the captured graph when ``use_graph``), everything else through prefill kernels as a
+        ragged batch of portions.  After a call that asked for a slot's last place, ``decode_step`` can carry on greedily."""
+        if self.heartbeat is not None:
+            self.heartbeat.check_fast()
+        slots = [e[0] for e in entries]
+        if len(set(slots)) != len(slots) or any(not 0 <= s < self.batch for s in slots):
+            raise ValueError(f"slots {slots} of a batch of {self.batch}")
+        norm = []
+        for slot, toks, want in entries:
+            toks = torch.as_tensor(toks, dtype=torch.int64).reshape(-1)
+            n = toks.numel()
+            if n < 1 or self._lens[slot] + n > self._admitted:
+                raise ValueError(f"{n} tokens after {self._lens[slot]} do not fit the {self._admitted} admitted per sequence")
+            if any(not 0 <= w < n for w in want):
+                raise ValueError(f"wanted places {list(want)} of a portion of {n} tokens")
+            norm.append((slot, toks, list(want)))
+        if not norm:
+            return []
+        if all(t.numel() == 1 and self._lens[s] > 0 for s, t, _ in norm):
+            return self._step_decode(norm, use_graph)
+        return self._extend(norm)
+
+    def _step_decode(self, entries, use_graph: bool) -> list[torch.Tensor]:
+        mine = {s for s, _, _ in entries}
+        others = [b for b in range(self.batch) if b not in mine and self._lens[b] > 0]
+        keep = self.tokens.clone() if others else None         # their next token is not this step's business
+        idx = torch.tensor([s for s, _, _ in entries], dtype=torch.int64).to(self.device, non_blocking=True)
+        self.tokens.index_copy_(0, idx, torch.cat([t for _, t, _ in entries]).to(self.device, non_blocking=True))
+        self._advance(mine, use_graph)
+        if keep is not None:
+            oi = torch.tensor(others, dtype=torch.int64).to(self.device, non_blocking=True)
+            self.tokens.index_copy_(0, oi, keep.index_select(0, oi))
+        logits = self._graph_logits[self.batch] if use_graph else self.model.last_logits
+        return [logits[s:s + 1][:len(w)].float().repeat(len(w), 1) if w else logits.new_empty((0, logits.shape[1]), dtype=torch.float32)
+                for s, _, w in entries]
+
+    def _extend(self, entries) -> list[torch.Tensor]:
+        """Portions of any length for any set of slots; long ones are cut so that a call carries at most
+        ``rt.max_prefill_tokens`` tokens, and pages nobody can see any more are given back in between."""
+        cap = self.rt.max_prefill_tokens
+        if not self.model.supports_portions and any(self._lens[s] > 0 or t.numel() > cap for s, t, _ in entries):
+            raise ValueError("this model's prefill takes whole prompts only")
+        dev = self.device
+        out = [torch.empty((len(w), self.cfg.vocab), dtype=torch.float32, device=dev) for _, _, w in entries]
+        done = [0] * len(entries)
+        while True:
+            room, part = cap, []                    # (entry, first token, tokens)
+            for i, (s, t, _) in enumerate(entries):
+                n = min(t.numel() - done[i], room)
+                if n > 0 and (self.model.supports_portions or n == t.numel()):
+                    part.append((i, done[i], n))
+                    room -= n
+            if not part:
+                break
+            ids, pos, sid, cu, rows, got = [], [], [], [0], [], []
+            for i, a, n in part:
+                slot, toks, want = entries[i]
+                start = self._lens[slot]
+                self.kv.retire(slot, start)
+                self.kv.admit(slot, start + n)
+                ids.append(toks[a:a + n])
+                pos.append(torch.arange(start, start + n, dtype=torch.int32))
+                sid.append(torch.full((n,), slot, dtype=torch.int32))
+                here = [k for k, w in enumerate(want) if a <= w < a + n]
+                if here:
+                    got.append((i, here, len(rows), next((len(rows) + j for j, k in enumerate(here) if want[k] == toks.numel() - 1), None)))
+                    rows += [cu[-1] + want[k] - a for k in here]
+                cu.append(cu[-1] + n)
+                self._lens[slot] = start + n
+                done[i] = a + n
+            self.kv.flush()
+            last = torch.tensor(rows if rows or self.model.supports_portions else [0], dtype=torch.int64)
+            nxt = self.model.forward(torch.cat(ids).to(dev, non_blocking=True), torch.cat(pos).to(dev, non_blocking=True), self.kv,
+                                     mode="prefill", cu_seqlens=torch.tensor(cu, dtype=torch.int32).to(dev, non_blocking=True),
+                                     max_len=max(n for _, _, n in part), seq_ids=torch.cat(sid).to(dev, non_blocking=True),
+                                     last_idx=last.to(dev, non_blocking=True))
+            default_workspace(dev).next_step()
+            for i, ks, r0, final in got:
+                out[i].index_copy_(0, torch.tensor(ks, dtype=torch.int64).to(dev, non_blocking=True),
+                                   self.model.last_logits[r0:r0 + len(ks)].float())
+                if final is not None:                    # the portion's last token was asked for: its greedy continuation
+                    self.tokens[entries[i][0]:entries[i][0] + 1].copy_(nxt[final:final + 1])
+        for slot, _, _ in entries:
+            n = self._lens[slot]
+            self.positions[slot:slot + 1].fill_(n)
+            self.kv.seq_lens[slot:slot + 1].fill_(n + 1)
+            self.active[slot:slot + 1].fill_(1)
+            self._active_host[slot] = 1
+        self._host_len = max(self._lens)
+        return out
 
     def admit_sequence(self, slot: int, prompt: torch.Tensor, use_graph: bool = True) -> torch.Tensor:
         """Between two decode steps: put a new sequence into slot ``slot`` (empty, or whose sequence is finished) of the
@@ -231,13 +355,17 @@ class Engine:
         S = int(prompt.numel())
         if S < 1 or S + 1 > self._admitted:
             raise ValueError(f"a prompt of {S} tokens does not fit the {self._admitted} admitted tokens")
-        self.kv.release(slot)
+        self._reset_slot(slot)
+        if S > self.rt.max_prefill_tokens and self.model.supports_portions:
+            self._extend([(slot, prompt.reshape(-1).cpu(), [S - 1])])
+            return self.tokens[slot:slot + 1].clone()
         self.kv.admit(slot, S + 1)
         self.kv.flush()
         self._prefill_equal(prompt.reshape(1, S).to(torch.int64).to(self.device, non_blocking=True), slot, use_graph)
         self.positions[slot:slot + 1].fill_(S)
         self.kv.seq_lens[slot:slot + 1].fill_(S + 1)
         self.active[slot:slot + 1].fill_(1)
+        self._active_host[slot] = 1
         self._lens[slot] = S
         self._host_len = max(self._lens)
         return self.tokens[slot:slot + 1].clone()
@@ -250,6 +378,7 @@ class Engine:
         self.positions[slot:slot + 1].zero_()
         self.kv.seq_lens[slot:slot + 1].zero_()
         self.active[slot:slot + 1].zero_()
+        self._active_host[slot] = 0
         self.tokens[slot:slot + 1].zero_()
         self._lens[slot] = 0
         self._host_len = max(self._lens)
@@ -283,17 +412,31 @@ class Engine:
         the kernels would refuse the write as well (status word), but the host knows first."""
         if self.heartbeat is not None:
             self.heartbeat.check_fast()
-        if self._host_len + 1 > self._admitted:
-            raise RuntimeError(f"decode step at position {self._host_len} exceeds the {self._admitted} tokens per "
+        return self._advance(None, use_graph)
+
+    def _advance(self, slots, use_graph: bool) -> torch.Tensor:
+        """One decode step of the sequences in ``slots`` (None: all that run); the others stay where they are."""
+        run = [b for b, n in enumerate(self._lens) if n > 0 and (slots is None or b in slots)]
+        top = max((self._lens[b] for b in run), default=self._host_len)
+        if top + 1 > self._admitted:
+            raise RuntimeError(f"decode step at position {top} exceeds the {self._admitted} tokens per "
                                f"sequence admitted by start_batch")
         # this step writes token number len + 1 of every running sequence: take the page it lands on if the sequence
-        # does not own it yet (once per page_size steps and sequence), and push the page table if a row changed
-        for b, n in enumerate(self._lens):
-            if n > 0:
-                self.kv.admit(b, n + 1)
-                self._lens[b] = n + 1
+        # does not own it yet (once per page_size steps and sequence), give back what no layer can see any more, and
+        # push the page table if a row changed
+        for b in run:
+            n = self._lens[b]
+            self.kv.retire(b, n)
+            self.kv.admit(b, n + 1)
+            self._lens[b] = n + 1
+        want = [0] * self.batch
+        for b in run:
+            want[b] = 1
+        if want != self._active_host:
+            self.active.copy_(torch.tensor(want, dtype=torch.int32), non_blocking=True)
+            self._active_host = want
+        self._host_len = max(self._lens)
         self.kv.flush()
-        self._host_len += 1
         if not use_graph:
             self._decode_body()
             return self.tokens
@@ -316,6 +459,7 @@ class Engine:
             self.kernels_per_step = _lib.LAUNCHES[0] - n0      # this library's kernels inside one replay
             self.tokens.copy_(saved[0]); self.positions.copy_(saved[1]); self.kv.seq_lens.copy_(saved[2])
             self._graphs[self.batch] = g
+            self._graph_logits[self.batch] = getattr(self.model, "last_logits", None)
         with op_range(f"decode_step.bs{self.batch}"):
             g.replay()
         return self.tokens
@@ -330,6 +474,7 @@ class Engine:
             self.heartbeat = None
         torch.cuda.synchronize(self.device)
         self._graphs.clear()
+        self._graph_logits.clear()
         self._prefill_graphs.clear()
         self._prefill_pool = None
         self.model._decode_scratch.clear()

@@ -12,6 +12,16 @@ from dataclasses import asdict, dataclass, field, replace
 
 
 @dataclass(frozen=True)
+class CacheSpec:
+    """What one layer (one pass of it, if layers repeat) keeps per token in the paged cache."""
+    kv_heads: int
+    dk: int                       # stored key size per head
+    dv: int                       # stored value size per head
+    dtype: str = "bfloat16"
+    chunk: int | None = None      # positions only see their own block of this many positions; None: all earlier ones
+
+
+@dataclass(frozen=True)
 class ModelConfig:
     name: str
     n_layers: int
@@ -33,6 +43,9 @@ class ModelConfig:
     @property
     def is_moe(self) -> bool:
         return self.n_experts > 0
+
+    def cache_layout(self, rt: "RuntimeConfig") -> list[CacheSpec]:
+        return [CacheSpec(kv_heads_per_rank(self, rt.tp), self.head_dim, self.head_dim)] * self.n_layers
 
     def to_json(self) -> str:
         return json.dumps(asdict(self))
@@ -89,6 +102,8 @@ class RuntimeConfig:
     max_seq_len: int = 2048
     max_prefill_tokens: int = 32768     # most tokens one prefill call may carry (sizes the symmetric TP buffers)
     fused_collectives: bool = True      # in-kernel peer-memory collectives; False = NCCL between kernels
+    dtype: str = "bfloat16"             # "float32": everything in 32-bit (families that have such a form)
+    kv_pool_tokens: int = 0             # tokens all sequences together may hold in the cache; 0: every slot its maximum
     wait_limit_ms: int = 2000           # bound of every device-side wait
     debug: bool = False
 

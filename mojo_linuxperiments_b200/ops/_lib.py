@@ -17,16 +17,18 @@ import os
 
 
 def _variant() -> str:
-    """Which build of the kernel library this process loads: B200RT_KERNELS=trace (in-kernel time stamps) or debug
-    (range-checked peer / scratch accesses); B200RT_DEBUG=1 also selects the debug build.  Default: production."""
+    """Which build of the kernel library this process loads: B200RT_KERNELS=trace (in-kernel time stamps), debug
+    (range-checked peer / scratch accesses) or dense (only the kernels of the unquantised models); B200RT_DEBUG=1 also
+    selects the debug build.  Default: production."""
     v = os.environ.get("B200RT_KERNELS", "").strip().lower()
-    if v in ("trace", "debug"):
+    if v in ("trace", "debug", "dense"):
         return v
     return "debug" if os.environ.get("B200RT_DEBUG", "0") not in ("", "0") else ""
 
 
-_LIB_PATH = Path(__file__).resolve().parent.parent / "_lib" / (
-    "libb200_kernels.so" if not _variant() else f"libb200_kernels_{_variant()}.so")
+def _lib_path() -> Path:
+    v = _variant()
+    return Path(__file__).resolve().parent.parent / "_lib" / ("libb200_kernels.so" if not v else f"libb200_kernels_{v}.so")
 
 
 class KernelError(RuntimeError):
@@ -35,17 +37,21 @@ class KernelError(RuntimeError):
 
 @lru_cache(maxsize=None)
 def lib() -> ctypes.CDLL:
-    if not _LIB_PATH.exists():
+    path = _lib_path()
+    if not path.exists():
         raise KernelError(
-            f"{_LIB_PATH} is missing: run `python -m mojo_linuxperiments_b200._build --all` (needs nvcc, no GPU)")
-    L = ctypes.CDLL(str(_LIB_PATH))
+            f"{path} is missing: run `python -m mojo_linuxperiments_b200._build --all` (needs nvcc, no GPU)")
+    L = ctypes.CDLL(str(path))
+    subset = _variant() == "dense"          # a part of the library: what it does not have is an error where it is called
     for name in dir(_Sig):
         if name.startswith("b200_"):
             restype, argtypes = getattr(_Sig, name)
             try:
                 fn = getattr(L, name)
             except AttributeError as e:  # stale library
-                raise KernelError(f"{name} not found in {_LIB_PATH}; rebuild the kernel library") from e
+                if subset:
+                    continue
+                raise KernelError(f"{name} not found in {path}; rebuild the kernel library") from e
             fn.restype = restype
             fn.argtypes = argtypes
     return L
@@ -91,6 +97,15 @@ class _Sig:
     b200_rope_kv_write = (I, [P, LL, P, P, P, P, P, P, F, P, P, P, P, P, I, I, I, I, I, I, I, P, P])
     b200_embed_gather = (I, [P, P, P, I, I, I, P])
     b200_argmax_rows = (I, [P, LL, I, I, I, I, P, P, P])
+    b200_argmax_rows_f32 = (I, [P, LL, I, I, I, I, P, P, P])
+    b200_bf16_gemm = (I, [P, LL, P, LL, I, I, I, P, P, I, I, P])
+    b200_bf16_gemm_decode = (I, [P, LL, P, LL, I, I, I, P, P, I, I, P])
+    b200_f32_gemm = (I, [P, LL, P, LL, I, I, I, P, P])
+    b200_rotary_paged = (I, [P, LL, I, I, P, P, P, P, I, I, I, P, P, P])
+    b200_embed_norm = (I, [P, P, LL, I, I, F, I, I, P, P, P, P])
+    b200_attn_paged = (I, [P, LL, P, LL, I, I, P, P, P, P, P, P, P])
+    b200_attn_prefill_paged = (I, [P, LL, P, LL, I, I, I, I, P, P, P, P, P, P, P])
+    b200_attn_decode_paged = (I, [P, LL, P, LL, I, I, P, P, P, P, I, I, I, P, P, I, P, P])
     b200_argmax_merge = (I, [P, P, I, I, P, P])
     b200_attn_decode_scratch_floats = (c_size_t, [I, I, I])
     b200_attn_decode = (I, [P, P, P, P, P, P, P, I, I, I, I, I, I, F, P, P])
@@ -110,6 +125,24 @@ class QuantProlog(ctypes.Structure):
     _fields_ = [("mode", c_int), ("x", c_void_p), ("ldx", c_longlong), ("residual", c_void_p), ("ldr", c_longlong),
                 ("gamma", c_void_p), ("eps", c_float), ("q", c_void_p), ("scale", c_void_p), ("flags", c_void_p),
                 ("step", c_void_p), ("residual_out", c_void_p), ("ldro", c_longlong), ("allow_inline", c_int)]
+
+
+class DenseEpilogue(ctypes.Structure):
+    """``b200_dense_epilogue`` of csrc/kernels/api.h: what a dense linear does with its result."""
+    _fields_ = [("mode", c_int), ("out_f32", c_int), ("exact", c_int), ("y", c_void_p), ("ldy", c_longlong), ("x", c_void_p),
+                ("ldx", c_longlong), ("add", c_void_p), ("mult", c_float), ("norm_w", c_void_p), ("norm_b", c_void_p),
+                ("norm_alpha", c_float), ("limit", c_float)]
+
+
+class PagedCacheDesc(ctypes.Structure):
+    """``b200_paged_cache`` of csrc/kernels/api.h."""
+    _fields_ = [("data", c_void_p), ("f32", c_int), ("kv_heads", c_int), ("page_size", c_int), ("dk", c_int), ("dv", c_int),
+                ("num_pages", c_int), ("page_table", c_void_p), ("num_seqs", c_int), ("max_pages", c_int)]
+
+
+class AttnSpecDesc(ctypes.Structure):
+    """``b200_attn_spec`` of csrc/kernels/api.h."""
+    _fields_ = [("scale", c_float), ("chunk", c_int), ("sink", c_void_p), ("gate", c_void_p), ("ldg", c_longlong)]
 
 
 def ptr(t: torch.Tensor | None) -> int | None:

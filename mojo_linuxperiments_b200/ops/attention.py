@@ -1,6 +1,7 @@
 """RoPE + paged-KV write, prefill (tcgen05) and decode (split-KV) attention, embedding gather, greedy argmax."""
 from __future__ import annotations
 
+import ctypes
 import math
 
 import torch
@@ -11,21 +12,56 @@ from .workspace import default_workspace
 HEAD_DIM = 128
 
 
-def rope_tables(max_pos: int, theta: float, device, head_dim: int = HEAD_DIM):
-    """cos/sin tables [max_pos, head_dim/2] fp32 for the rotate-half convention (pairs i, i + head_dim/2)."""
-    inv = 1.0 / (theta ** (torch.arange(0, head_dim, 2, dtype=torch.float64) / head_dim))
+def rope_frequencies(dims: int, base: float, yarn=None):
+    """fp64 rotation frequency of each of the dims/2 pairs, and the factor on cos and sin.
+
+    ``yarn`` (factor, original, fast, slow): pairs that turn more than ``fast`` times within ``original`` positions keep
+    their frequency, those that turn less than ``slow`` times are slowed down by ``factor``, with a linear ramp over
+    the pair index in between; the rotated vectors grow by 0.1 ln(factor) + 1."""
+    inv = float(base) ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
+    if yarn is None:
+        return inv, 1.0
+    n_pairs_log = 2.0 * math.log(base)
+
+    def pair_with(turns: float) -> float:
+        return dims * math.log(yarn.original / (2.0 * math.pi * turns)) / n_pairs_log
+    lo = max(math.floor(pair_with(yarn.fast)), 0)
+    hi = min(math.ceil(pair_with(yarn.slow)), dims - 1)
+    ramp = ((torch.arange(dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return inv / yarn.factor * ramp + inv * (1.0 - ramp), 0.1 * math.log(yarn.factor) + 1.0
+
+
+def rope_tables(max_pos: int, theta: float, device, head_dim: int = HEAD_DIM, yarn=None):
+    """cos/sin tables [max_pos, head_dim/2] fp32, one column per rotated pair (which two dimensions form a pair is the
+    kernel's business); with ``yarn`` the scaled frequencies and the factor on both tables."""
+    inv, mag = rope_frequencies(head_dim, theta, yarn)
     ang = torch.arange(max_pos, dtype=torch.float64)[:, None] * inv[None, :]
-    return ang.cos().float().to(device).contiguous(), ang.sin().float().to(device).contiguous()
+    return (ang.cos() * mag).float().to(device).contiguous(), (ang.sin() * mag).float().to(device).contiguous()
 
 
 class PagedKVCache:
-    """One layer's paged KV storage: [num_pages][2][kv_heads][page_size][128] bf16."""
+    """One layer's paged KV storage, one record per page: [kv_heads][page_size][dk] keys, then
+    [kv_heads][page_size][dv] values (bf16, or fp32 for the 32-bit form of a model)."""
 
-    def __init__(self, num_pages: int, kv_heads: int, page_size: int, device, storage: torch.Tensor | None = None):
-        shape = (num_pages, 2, kv_heads, page_size, HEAD_DIM)
-        self.data = storage if storage is not None else torch.zeros(shape, dtype=torch.bfloat16, device=device)
-        assert tuple(self.data.shape) == shape
-        self.num_pages, self.kv_heads, self.page_size = num_pages, kv_heads, page_size
+    def __init__(self, num_pages: int, kv_heads: int, page_size: int, device, storage: torch.Tensor | None = None,
+                 dk: int = HEAD_DIM, dv: int = HEAD_DIM, dtype: torch.dtype = torch.bfloat16):
+        shape = (num_pages, 2, kv_heads, page_size, dk) if dk == dv else (num_pages, kv_heads * page_size * (dk + dv))
+        self.data = storage.view(shape) if storage is not None else torch.zeros(shape, dtype=dtype, device=device)
+        self.num_pages, self.kv_heads, self.page_size, self.dk, self.dv = num_pages, kv_heads, page_size, dk, dv
+
+    def keys(self) -> torch.Tensor:
+        """[num_pages][kv_heads][page_size][dk] view"""
+        n = self.kv_heads * self.page_size * self.dk
+        return self.data.view(self.num_pages, -1)[:, :n].unflatten(1, (self.kv_heads, self.page_size, self.dk))
+
+    def values(self) -> torch.Tensor:
+        n = self.kv_heads * self.page_size * self.dk
+        return self.data.view(self.num_pages, -1)[:, n:].unflatten(1, (self.kv_heads, self.page_size, self.dv))
+
+    def desc(self, page_table: torch.Tensor) -> "_lib.PagedCacheDesc":
+        return _lib.PagedCacheDesc(self.data.data_ptr(), 1 if self.data.dtype == torch.float32 else 0, self.kv_heads,
+                                   self.page_size, self.dk, self.dv, self.num_pages, page_table.data_ptr(),
+                                   page_table.shape[0], page_table.shape[1])
 
 
 def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, hq: int, hkv: int, *,
@@ -260,16 +296,17 @@ def embed_gather(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor | Non
 
 
 def argmax_rows(logits: torch.Tensor, index_offset: int = 0, chunks: int | None = None):
-    """Candidates (max value fp32, index int64 + offset) per row of bf16 logits [rows, n], one per column chunk:
+    """Candidates (max value fp32, index int64 + offset) per row of bf16 or fp32 logits [rows, n], one per column chunk:
     returns ([chunks, rows], [chunks, rows]); ``argmax_merge`` picks the winner (lowest index wins ties)."""
     rows, n = logits.shape
-    assert logits.dtype == torch.bfloat16 and logits.stride(1) == 1
+    assert logits.dtype in (torch.bfloat16, torch.float32) and logits.stride(1) == 1
     if chunks is None:
         chunks = max(1, min(64, n // 2048, 296 // max(rows, 1) + 1))
     out_val = torch.empty((chunks, rows), dtype=torch.float32, device=logits.device)
     out_idx = torch.empty((chunks, rows), dtype=torch.int64, device=logits.device)
-    _lib.check(_lib.lib().b200_argmax_rows(logits.data_ptr(), logits.stride(0), rows, n, index_offset, chunks,
-                                           out_val.data_ptr(), out_idx.data_ptr(), _lib.stream()), "argmax_rows")
+    fn = _lib.lib().b200_argmax_rows if logits.dtype == torch.bfloat16 else _lib.lib().b200_argmax_rows_f32
+    _lib.check(fn(logits.data_ptr(), logits.stride(0), rows, n, index_offset, chunks,
+                  out_val.data_ptr(), out_idx.data_ptr(), _lib.stream()), "argmax_rows")
     return out_val, out_idx
 
 
@@ -284,3 +321,88 @@ def argmax_merge(cand_val: torch.Tensor, cand_idx: torch.Tensor, out_idx: torch.
     _lib.check(_lib.lib().b200_argmax_merge(cand_val.data_ptr(), cand_idx.data_ptr(), world, rows, out_idx.data_ptr(),
                                             _lib.stream()), "argmax_merge")
     return out_idx
+
+
+# ---------------------------------------------------------------------------------------------------------
+# attention over the paged cache with free head sizes (bf16 or fp32), optional chunk mask, sink and output gate
+# ---------------------------------------------------------------------------------------------------------
+TC_HEAD_DIM = 128              # largest key / value size of the tensor-core prefill kernel
+DECODE_HEAD_DIM = 256          # ... of the one-launch decode kernel
+PAGE = 16                      # page size of both
+
+
+def attn_spec(scale: float, *, chunk: int | None = None, sink: torch.Tensor | None = None, gate: torch.Tensor | None = None):
+    """``chunk``: a position sees only its own block of that many positions; ``sink`` fp32 [hq]: one more exponent per head
+    in the softmax's denominator; ``gate`` [M, hq] (row stride free): logits of a sigmoid on each head's output."""
+    if sink is not None:
+        assert sink.dtype == torch.float32 and sink.is_contiguous()
+    return _lib.AttnSpecDesc(float(scale), int(chunk or 0), _lib.ptr(sink), _lib.ptr(gate), gate.stride(0) if gate is not None else 0)
+
+
+def rotary_paged(qkv: torch.Tensor, hq: int, positions: torch.Tensor, seq_ids: torch.Tensor | None, cos: torch.Tensor | None,
+                 sin: torch.Tensor | None, cache: PagedKVCache, page_table: torch.Tensor, *, interleaved: bool = True) -> None:
+    """qkv [M, hq dk + kv_heads (dk + dv) (+ more)]: q is rotated in place, k (rotated) and v are appended to ``cache``."""
+    assert qkv.dtype == cache.data.dtype and qkv.stride(1) == 1 and positions.dtype == torch.int32 and page_table.dtype == torch.int32
+    rc = _lib.lib().b200_rotary_paged(
+        qkv.data_ptr(), qkv.stride(0), hq, qkv.shape[0], positions.data_ptr(), _lib.ptr(seq_ids), _lib.ptr(cos), _lib.ptr(sin),
+        cos.shape[1] if cos is not None else 0, 1 if interleaved else 0, cos.shape[0] if cos is not None else 1 << 30,
+        ctypes.byref(cache.desc(page_table)), default_workspace(qkv.device).status.data_ptr(), _lib.stream())
+    _lib.check(rc, "rotary_paged")
+
+
+def attn_paged(q: torch.Tensor, hq: int, positions: torch.Tensor, seq_ids: torch.Tensor | None, cache: PagedKVCache,
+               page_table: torch.Tensor, spec, out: torch.Tensor, seq_lens: torch.Tensor | None = None) -> torch.Tensor:
+    """General form: rows of q (already rotated; [M, hq dk], row stride free) against the cached keys of their sequence."""
+    assert q.dtype == cache.data.dtype == out.dtype and q.stride(1) == 1 and out.stride(1) == 1
+    rc = _lib.lib().b200_attn_paged(
+        q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), hq, q.shape[0], positions.data_ptr(), _lib.ptr(seq_ids),
+        _lib.ptr(seq_lens), ctypes.byref(cache.desc(page_table)), ctypes.byref(spec), default_workspace(q.device).status.data_ptr(),
+        _lib.stream())
+    _lib.check(rc, "attn_paged")
+    return out
+
+
+def attn_prefill_paged(q: torch.Tensor, hq: int, positions: torch.Tensor, seq_ids: torch.Tensor, cu_seqlens: torch.Tensor,
+                       max_len: int, cache: PagedKVCache, page_table: torch.Tensor, spec, out: torch.Tensor) -> torch.Tensor:
+    """Portions of sequences (rows cu[b] .. cu[b+1] are consecutive positions, keys in the cache already): tensor cores for
+    bf16 heads of up to 128, the general kernel otherwise."""
+    if cache.data.dtype != torch.bfloat16 or max(cache.dk, cache.dv) > TC_HEAD_DIM or cache.page_size != PAGE:
+        return attn_paged(q, hq, positions, seq_ids, cache, page_table, spec, out)
+    rc = _lib.lib().b200_attn_prefill_paged(
+        q.data_ptr(), q.stride(0), out.data_ptr(), out.stride(0), hq, q.shape[0], cu_seqlens.numel() - 1, int(max_len),
+        cu_seqlens.data_ptr(), positions.data_ptr(), _lib.ptr(seq_ids), ctypes.byref(cache.desc(page_table)), ctypes.byref(spec),
+        default_workspace(q.device).status.data_ptr(), _lib.stream())
+    _lib.check(rc, "attn_prefill_paged")
+    return out
+
+
+def pick_decode_splits_paged(B: int, kv_groups: int, max_keys: int, num_sms: int = 148) -> int:
+    """CTAs per (sequence, KV head): enough to fill the GPU, at least 64 keys (one page per warp) each, one cluster at most."""
+    pairs = max(1, B * kv_groups)
+    cap = max(1, min(8, max_keys // 64))
+    s = 1
+    while s < cap and pairs * s < 2 * num_sms:
+        s *= 2
+    return min(s, cap)
+
+
+def attn_decode_paged(qkv: torch.Tensor, hq: int, positions: torch.Tensor, seq_lens: torch.Tensor, cos: torch.Tensor | None,
+                      sin: torch.Tensor | None, cache: PagedKVCache, page_table: torch.Tensor, spec, out: torch.Tensor, *,
+                      interleaved: bool = True, splits: int | None = None) -> torch.Tensor:
+    """One new token per sequence slot (row b = slot b): rotary embedding, cache append, attention, sink and gate.  One
+    launch for bf16 heads of up to 256; otherwise ``rotary_paged`` + ``attn_paged``."""
+    B = qkv.shape[0]
+    if cache.data.dtype != torch.bfloat16 or max(cache.dk, cache.dv) > DECODE_HEAD_DIM or cache.page_size != PAGE:
+        rotary_paged(qkv, hq, positions, None, cos, sin, cache, page_table, interleaved=interleaved)
+        return attn_paged(qkv, hq, positions, None, cache, page_table, spec, out, seq_lens=seq_lens)
+    if splits is None:
+        keys = page_table.shape[1] * cache.page_size
+        groups = cache.kv_heads * ((hq // cache.kv_heads + 15) // 16)
+        splits = pick_decode_splits_paged(B, groups, min(keys, spec.chunk) if spec.chunk > 0 else keys, _lib.num_sms(qkv.device.index))
+    rc = _lib.lib().b200_attn_decode_paged(
+        qkv.data_ptr(), qkv.stride(0), out.data_ptr(), out.stride(0), hq, B, positions.data_ptr(), seq_lens.data_ptr(),
+        _lib.ptr(cos), _lib.ptr(sin), cos.shape[1] if cos is not None else 0, 1 if interleaved else 0,
+        cos.shape[0] if cos is not None else 1 << 30, ctypes.byref(cache.desc(page_table)), ctypes.byref(spec), splits,
+        default_workspace(qkv.device).status.data_ptr(), _lib.stream())
+    _lib.check(rc, "attn_decode_paged")
+    return out
