@@ -69,7 +69,8 @@ struct DpShape {
   static constexpr int SMEM = (RING > MERGE ? RING : MERGE) + QBYTES + 128;
 };
 
-template <int DK, int DV, int STG>
+// FULL: dk == DK and dv == DV, so the MMA steps and the copies unroll without conditions
+template <int DK, int DV, int STG, bool FULL>
 __global__ void __launch_bounds__(DP_THREADS)
 attn_decode_paged_kernel(const __grid_constant__ DecodePagedParams p) {
   using Sh = DpShape<DK, DV, STG>;
@@ -82,7 +83,7 @@ attn_decode_paged_kernel(const __grid_constant__ DecodePagedParams p) {
   const int rank = blockIdx.x, S = p.splits, b = blockIdx.z;
   const int kvh = blockIdx.y / p.hgroups, hg = blockIdx.y - kvh * p.hgroups;
   const int group = p.hq / p.c.kv_heads, g0 = hg * 16, G = min(16, group - g0), h0 = kvh * group + g0;
-  const int dk = p.c.dk, dv = p.c.dv, ksteps = (dk + 15) >> 4, vsteps = (dv + 15) >> 4;
+  const int dk = FULL ? DK : p.c.dk, dv = FULL ? DV : p.c.dv, ksteps = (dk + 15) >> 4, vsteps = (dv + 15) >> 4;
   const int pos = p.positions[b];
   const bool empty = p.seq_lens[b] <= 0;
   const bool bad = pos < 0 || pos >= p.max_pos || pos / DP_PS >= p.c.max_pages;
@@ -108,22 +109,49 @@ attn_decode_paged_kernel(const __grid_constant__ DecodePagedParams p) {
   if (dk & 15)
     for (int i = lane; i < STG * 16; i += 32)
       *reinterpret_cast<uint4*>(ring + (i >> 4) * Sh::STAGE + ((i & 15) * Sh::KP + dk) * 2) = make_uint4(0u, 0u, 0u, 0u);
+  // Page ids of this warp's next 32 pages sit in its lanes, so that a request never waits for a table look-up; the
+  // (row, 16-byte column) of a lane's first copy and its step to the next one avoid divisions.
+  const int kc = dk >> 3, vc = dv >> 3;
+  const int kr0 = lane / kc, kc0 = lane - kr0 * kc, krs = 32 / kc, kcs = 32 - krs * kc;
+  const int vr0 = lane / vc, vc0 = lane - vr0 * vc, vrs = 32 / vc, vcs = 32 - vrs * vc;
+  int ids = 0, ids_from = -32;
   auto issue = [&](int i) {
     if (i < mine) {
+      if (i >= ids_from + 32) {
+        ids_from = i;
+        ids = i + lane < mine ? pt[ta + warp + (i + lane) * DP_WARPS] : 0;
+      }
       const int t = ta + warp + i * DP_WARPS;
-      const int page = pt[t];
+      const int page = __shfl_sync(0xffffffffu, ids, i - ids_from);
       const bool page_ok = page >= 0 && page < p.c.num_pages;
       const __nv_bfloat16* src = cache + (page_ok ? static_cast<size_t>(page) * rec : 0);
       const uint32_t kd = smem_u32(ring + (i % STG) * Sh::STAGE), vd = kd + 16 * Sh::KP * 2;
       const int left = page_ok ? pos - t * DP_PS : 0;           // rows of this page before the new token
-      const int kc = dk >> 3, vc = dv >> 3;
-      for (int u = lane; u < 16 * kc; u += 32) {
-        const int r = u / kc, c = u - r * kc;
-        dp_cp16(kd + (r * Sh::KP + c * 8) * 2, src + k_off + u * 8, r < left);
+      const __nv_bfloat16* ks = src + k_off + lane * 8;
+      const __nv_bfloat16* vs = src + v_off + lane * 8;
+      if constexpr (FULL) {
+#pragma unroll
+        for (int u = 0; u < DK / 16; ++u) {
+          const int r = kr0 + u * (256 / DK);
+          dp_cp16(kd + (r * Sh::KP + kc0 * 8) * 2, ks + u * 256, r < left);
+        }
+#pragma unroll
+        for (int u = 0; u < DV / 16; ++u) {
+          const int r = vr0 + u * (256 / DV);
+          dp_cp16(vd + (r * Sh::VP + vc0 * 8) * 2, vs + u * 256, r < left);
+        }
+        dp_commit();
+        return;
       }
-      for (int u = lane; u < 16 * vc; u += 32) {
-        const int r = u / vc, c = u - r * vc;
-        dp_cp16(vd + (r * Sh::VP + c * 8) * 2, src + v_off + u * 8, r < left);
+      for (int r = kr0, c = kc0; r < 16; ks += 256) {
+        dp_cp16(kd + (r * Sh::KP + c * 8) * 2, ks, r < left);
+        r += krs; c += kcs;
+        if (c >= kc) { c -= kc; ++r; }
+      }
+      for (int r = vr0, c = vc0; r < 16; vs += 256) {
+        dp_cp16(vd + (r * Sh::VP + c * 8) * 2, vs, r < left);
+        r += vrs; c += vcs;
+        if (c >= vc) { c -= vc; ++r; }
       }
     }
     dp_commit();
@@ -161,7 +189,7 @@ attn_decode_paged_kernel(const __grid_constant__ DecodePagedParams p) {
   const uint32_t qaddr = smem_u32(qs) + (((lane & 7) + ((lane >> 3) & 1) * 8) * Sh::KP + (lane >> 4) * 8) * 2;
 #pragma unroll
   for (int kk = 0; kk < DK / 16; ++kk)
-    if (kk < ksteps) dp_ldm(qaddr + kk * 32, qa[kk]);
+    if (FULL || kk < ksteps) dp_ldm(qaddr + kk * 32, qa[kk]);
 
   float o[DV / 8][4];
 #pragma unroll
@@ -180,7 +208,7 @@ attn_decode_paged_kernel(const __grid_constant__ DecodePagedParams p) {
     const uint32_t ka = kd + (((lane & 7) + (lane >> 4) * 8) * Sh::KP + ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll
     for (int kk = 0; kk < DK / 16; ++kk)
-      if (kk < ksteps) {
+      if (FULL || kk < ksteps) {
         uint32_t kb[4];
         dp_ldm(ka + kk * 32, kb);
         dp_mma(s[0], qa[kk], kb[0], kb[1]);
@@ -223,7 +251,7 @@ attn_decode_paged_kernel(const __grid_constant__ DecodePagedParams p) {
     const uint32_t va = vd + (((lane & 7) + ((lane >> 3) & 1) * 8) * Sh::VP + (lane >> 4) * 8) * 2;
 #pragma unroll
     for (int n = 0; n < DV / 16; ++n)
-      if (n < vsteps) {
+      if (FULL || n < vsteps) {
         uint32_t vb[4];
         dp_ldm_t(va + n * 32, vb);
         dp_mma(o[2 * n], pa, vb[0], vb[1]);
@@ -323,17 +351,17 @@ attn_decode_paged_kernel(const __grid_constant__ DecodePagedParams p) {
   if (S > 1) cluster_sync_all();                 // no CTA leaves while a peer may still read its partials
 }
 
-template <int DK, int DV, int STG>
+template <int DK, int DV, int STG, bool FULL>
 static int launch_decode_paged(const DecodePagedParams& p, dim3 grid, cudaStream_t stream) {
   constexpr int SMEM = DpShape<DK, DV, STG>::SMEM;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_decode_paged_kernel<DK, DV, STG>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_paged_kernel<DK, DV, STG, FULL>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     if (e != cudaSuccess) return -1000 - static_cast<int>(e);
-    cudaFuncSetAttribute(attn_decode_paged_kernel<DK, DV, STG>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+    cudaFuncSetAttribute(attn_decode_paged_kernel<DK, DV, STG, FULL>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
     configured = true;
   }
-  launch_ex(attn_decode_paged_kernel<DK, DV, STG>, grid, dim3(DP_THREADS), SMEM, stream, p.splits, p);
+  launch_ex(attn_decode_paged_kernel<DK, DV, STG, FULL>, grid, dim3(DP_THREADS), SMEM, stream, p.splits, p);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -2000 - static_cast<int>(e);
 }
@@ -358,7 +386,9 @@ extern "C" int b200_attn_decode_paged(const void* qkv, long long ld, void* out, 
   p.sink = s->sink; p.gate = static_cast<const __nv_bfloat16*>(s->gate); p.ldg = s->ldg; p.splits = splits; p.status = status;
   const dim3 grid(splits, c->kv_heads * p.hgroups, B);
   const int d = c->dk > c->dv ? c->dk : c->dv;
-  if (d <= 64) return launch_decode_paged<64, 64, 6>(p, grid, stream);
-  if (d <= 128) return launch_decode_paged<128, 128, 3>(p, grid, stream);
-  return launch_decode_paged<256, 256, 3>(p, grid, stream);
+  if (c->dk == 64 && c->dv == 64) return launch_decode_paged<64, 64, 6, true>(p, grid, stream);
+  if (c->dk == 128 && c->dv == 128) return launch_decode_paged<128, 128, 3, true>(p, grid, stream);
+  if (d <= 64) return launch_decode_paged<64, 64, 6, false>(p, grid, stream);
+  if (d <= 128) return launch_decode_paged<128, 128, 3, false>(p, grid, stream);
+  return launch_decode_paged<256, 256, 3, false>(p, grid, stream);
 }

@@ -130,21 +130,41 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
     const int q = warp & 3;                 // TMEM lane quarter this warp may read
     float* piece = stage_f + (warp - 2) * 32 * BG_SP;
     int idx = 0;
+    const bool residual = p.epi.mode == B200_EPI_RESIDUAL;
+    const int rr0 = lane >> 3, c4 = (lane & 7) * 4;          // row group and column quad of this lane in a 32 x 32 piece
     for (int tile = blockIdx.x; tile < p.num_tiles; tile += gridDim.x, ++idx) {
       const int a = idx & 1;
       int m_tile, n_tile;
       bg_tile_coords(p, tile, m_tile, n_tile);
+      const int m0 = m_tile * 128 + q * 32, n0 = n_tile * BN;
+      // The residual rows of a piece are requested one piece ahead (the first even before the accumulator is complete):
+      // the epilogue is four warps, so what it needs is loads in flight.
+      float4 xn[8];
+      auto load_x = [&](int c) {
+        const int n = n0 + c * 32 + c4;
+#pragma unroll
+        for (int it = 0; it < 8; ++it) {
+          const int m = m0 + it * 4 + rr0;
+          if (m < p.M && n < p.N) xn[it] = *reinterpret_cast<const float4*>(p.epi.x + static_cast<long long>(m) * p.epi.ldx + n);
+        }
+      };
+      if (residual) load_x(0);
       // one verdict per warp: the lanes stay together at the TMEM loads
       const bool ok = __all_sync(0xffffffffu, mbar_wait(tfull_bar(a), (idx >> 1) & 1u, abort_flag, p.status, (ST_TIMEOUT_TMEM_FULL | (9 << 8)), limit));
       if (!ok) break;
       tc_fence_after();
       const uint32_t t_addr = tmem_base + (static_cast<uint32_t>(q * 32) << 16) + a * BN;
-      const int m0 = m_tile * 128 + q * 32, n0 = n_tile * BN;
 #pragma unroll 1
       for (int c = 0; c < BN / 32; ++c) {
         if (n0 + c * 32 >= p.N) break;
         uint32_t r[32];
         tmem_ld_x32(t_addr + c * 32, r);
+        float4 xc[8];
+        if (residual) {
+#pragma unroll
+          for (int it = 0; it < 8; ++it) xc[it] = xn[it];
+          if (c + 1 < BN / 32) load_x(c + 1);
+        }
         tmem_ld_wait();
         float* mine = piece + lane * BG_SP;
 #pragma unroll
@@ -152,11 +172,22 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
           *reinterpret_cast<float4*>(mine + 4 * g) = make_float4(__uint_as_float(r[4 * g]), __uint_as_float(r[4 * g + 1]),
                                                                  __uint_as_float(r[4 * g + 2]), __uint_as_float(r[4 * g + 3]));
         __syncwarp();
-        const int n = n0 + c * 32 + (lane & 7) * 4;
+        const int n = n0 + c * 32 + c4;
+        if (n < p.N) {
+          if (residual) {
+            const EpiNorm nw = epi_norm_columns(p.epi, n);
 #pragma unroll
-        for (int it = 0; it < 8; ++it) {
-          const int rr = it * 4 + (lane >> 3), m = m0 + rr;
-          if (m < p.M && n < p.N) epi_apply4(p.epi, m, n, *reinterpret_cast<const float4*>(piece + rr * BG_SP + (lane & 7) * 4));
+            for (int it = 0; it < 8; ++it) {
+              const int rr = it * 4 + rr0, m = m0 + rr;
+              if (m < p.M) epi_residual4(p.epi, nw, m, n, *reinterpret_cast<const float4*>(piece + rr * BG_SP + c4), xc[it]);
+            }
+          } else {
+#pragma unroll
+            for (int it = 0; it < 8; ++it) {
+              const int rr = it * 4 + rr0, m = m0 + rr;
+              if (m < p.M) epi_apply4(p.epi, m, n, *reinterpret_cast<const float4*>(piece + rr * BG_SP + c4));
+            }
+          }
         }
         __syncwarp();
       }

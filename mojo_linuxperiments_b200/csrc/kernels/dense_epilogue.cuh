@@ -40,16 +40,36 @@ __device__ __forceinline__ void store4_any(void* base, bool f32, long long off, 
   }
 }
 
-// element-wise norm of four residual values of columns n .. n+3
-__device__ __forceinline__ float4 epi_norm4(const b200_dense_epilogue& e, int n, float4 x, bool exact) {
-  const float4 w = __ldg(reinterpret_cast<const float4*>(e.norm_w + n));
-  const float4 b = __ldg(reinterpret_cast<const float4*>(e.norm_b + n));
+// weight and shift of the element-wise norm for columns n .. n+3 (zeros when the epilogue has none)
+struct EpiNorm { float4 w, b; };
+__device__ __forceinline__ EpiNorm epi_norm_columns(const b200_dense_epilogue& e, int n) {
+  EpiNorm k;
+  k.w = k.b = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (e.y) {
+    k.w = __ldg(reinterpret_cast<const float4*>(e.norm_w + n));
+    k.b = __ldg(reinterpret_cast<const float4*>(e.norm_b + n));
+  }
+  return k;
+}
+
+__device__ __forceinline__ float4 epi_norm4(const b200_dense_epilogue& e, const EpiNorm& k, float4 x, bool exact) {
   float4 o;
-  o.x = epi_tanh(e.norm_alpha * x.x, exact) * w.x + b.x;
-  o.y = epi_tanh(e.norm_alpha * x.y, exact) * w.y + b.y;
-  o.z = epi_tanh(e.norm_alpha * x.z, exact) * w.z + b.z;
-  o.w = epi_tanh(e.norm_alpha * x.w, exact) * w.w + b.w;
+  o.x = epi_tanh(e.norm_alpha * x.x, exact) * k.w.x + k.b.x;
+  o.y = epi_tanh(e.norm_alpha * x.y, exact) * k.w.y + k.b.y;
+  o.z = epi_tanh(e.norm_alpha * x.z, exact) * k.w.z + k.b.z;
+  o.w = epi_tanh(e.norm_alpha * x.w, exact) * k.w.w + k.b.w;
   return o;
+}
+
+// residual form with the old residual values `x` of row m, columns n .. n+3, already loaded
+__device__ __forceinline__ void epi_residual4(const b200_dense_epilogue& e, const EpiNorm& k, long long m, int n, float4 v, float4 x) {
+  x.x += e.mult * v.x; x.y += e.mult * v.y; x.z += e.mult * v.z; x.w += e.mult * v.w;
+  if (e.add) {
+    const float4 a = *reinterpret_cast<const float4*>(e.add + m * e.ldx + n);
+    x.x += a.x; x.y += a.y; x.z += a.z; x.w += a.w;
+  }
+  *reinterpret_cast<float4*>(e.x + m * e.ldx + n) = x;
+  if (e.y) store4_any(e.y, e.out_f32 != 0, m * e.ldy + n, epi_norm4(e, k, x, e.exact != 0));
 }
 
 // columns n .. n+3 (n a multiple of four, n < N) of row m
@@ -70,15 +90,7 @@ __device__ __forceinline__ void epi_apply4(const b200_dense_epilogue& e, long lo
       *reinterpret_cast<__nv_bfloat162*>(static_cast<__nv_bfloat16*>(e.y) + off) = __floats2bfloat162_rn(o0, o1);
     }
   } else {
-    float4* xp = reinterpret_cast<float4*>(e.x + m * e.ldx + n);
-    float4 x = *xp;
-    x.x += e.mult * v.x; x.y += e.mult * v.y; x.z += e.mult * v.z; x.w += e.mult * v.w;
-    if (e.add) {
-      const float4 a = *reinterpret_cast<const float4*>(e.add + m * e.ldx + n);
-      x.x += a.x; x.y += a.y; x.z += a.z; x.w += a.w;
-    }
-    *xp = x;
-    if (e.y) store4_any(e.y, f32, m * e.ldy + n, epi_norm4(e, n, x, e.exact != 0));
+    epi_residual4(e, epi_norm_columns(e, n), m, n, v, *reinterpret_cast<const float4*>(e.x + m * e.ldx + n));
   }
 }
 

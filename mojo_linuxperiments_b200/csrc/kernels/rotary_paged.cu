@@ -96,7 +96,7 @@ embed_norm_kernel(const long long* ids, const T* table, long long ldt, int vocab
     v.z = to_f(__ldg(table + id * ldt + n + 2)) * scale; v.w = to_f(__ldg(table + id * ldt + n + 3)) * scale;
     *reinterpret_cast<float4*>(x + m * e.ldx + n) = v;
     if (copy) *reinterpret_cast<float4*>(copy + m * e.ldx + n) = v;
-    if (e.y) store4_any(e.y, e.out_f32 != 0, m * e.ldy + n, epi_norm4(e, n, v, e.exact != 0));
+    if (e.y) store4_any(e.y, e.out_f32 != 0, m * e.ldy + n, epi_norm4(e, epi_norm_columns(e, n), v, e.exact != 0));
   }
 }
 

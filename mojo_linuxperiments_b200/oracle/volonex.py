@@ -73,9 +73,10 @@ def attention(h, mix: dict, m: dict):
     q = (h @ mix["q"].t()).view(T, H, d)
     k = (h @ mix["k"].t()).view(T, G, d)
     v = (h @ mix["v"].t()).view(T, G, dv)
-    pos = torch.arange(T, device=h.device)
-    freq, mag = yarn_frequencies(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
-    q, k = rotate_interleaved(q, pos, freq, mag), rotate_interleaved(k, pos, freq, mag)
+    if m.get("rot"):
+        pos = torch.arange(T, device=h.device)
+        freq, mag = yarn_frequencies(m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling"))
+        q, k = rotate_interleaved(q, pos, freq, mag), rotate_interleaved(k, pos, freq, mag)
     k, v = k.repeat_interleave(H // G, 1), v.repeat_interleave(H // G, 1)
     scores = torch.einsum("ihd,jhd->hij", q, k) * m["scale"]
     size = m["mask"]["size"] if m.get("mask") else None
