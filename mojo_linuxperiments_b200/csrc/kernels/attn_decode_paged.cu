@@ -140,18 +140,17 @@ attn_decode_paged_kernel(const __grid_constant__ DecodePagedParams p) {
           const int r = vr0 + u * (256 / DV);
           dp_cp16(vd + (r * Sh::VP + vc0 * 8) * 2, vs + u * 256, r < left);
         }
-        dp_commit();
-        return;
-      }
-      for (int r = kr0, c = kc0; r < 16; ks += 256) {
-        dp_cp16(kd + (r * Sh::KP + c * 8) * 2, ks, r < left);
-        r += krs; c += kcs;
-        if (c >= kc) { c -= kc; ++r; }
-      }
-      for (int r = vr0, c = vc0; r < 16; vs += 256) {
-        dp_cp16(vd + (r * Sh::VP + c * 8) * 2, vs, r < left);
-        r += vrs; c += vcs;
-        if (c >= vc) { c -= vc; ++r; }
+      } else {
+        for (int r = kr0, c = kc0; r < 16; ks += 256) {
+          dp_cp16(kd + (r * Sh::KP + c * 8) * 2, ks, r < left);
+          r += krs; c += kcs;
+          if (c >= kc) { c -= kc; ++r; }
+        }
+        for (int r = vr0, c = vc0; r < 16; vs += 256) {
+          dp_cp16(vd + (r * Sh::VP + c * 8) * 2, vs, r < left);
+          r += vrs; c += vcs;
+          if (c >= vc) { c -= vc; ++r; }
+        }
       }
     }
     dp_commit();

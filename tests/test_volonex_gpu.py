@@ -386,6 +386,13 @@ def uneven() -> LC.LayeredConfig:
     return LC.LayeredConfig("Volonex", 203, 108, layers, 2.5, 0.6, 1e-6, LC.Loop(1, 3, 3))
 
 
+def bare() -> LC.LayeredConfig:
+    """Odd sizes everywhere, the whole stack repeated, its last layer without feed-forward."""
+    a = LC.AttentionSpec(5, 5, 18, 22, 0.3, LC.Rotary(50.0, 18, LC.Yarn(2.0, 40.0, 4.0, 1.0)), 19)
+    b = LC.AttentionSpec(7, 1, 33, 9, 0.2, LC.Rotary(900.0, 6), 64)
+    return LC.LayeredConfig("Volonex", 131, 93, (LC.LayerSpec(a, LC.GatedMLP(51, 1.0)), LC.LayerSpec(b, None)), 1.7, 1.0, 1e-6, LC.Loop(0, 2, 2))
+
+
 def even(chunk=40, **kw) -> LC.LayeredConfig:
     kw = {"dim": 64, "vdim": 32, "rot_dims": 32, "base": 1e4, "scaling": LC.Yarn(2.0, 100.0, 8.0, 1.0), "limit": 1.5, "embed_scale": 3.0,
           "residual_mult": 0.8, **kw}
@@ -420,7 +427,7 @@ class Model:
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("make", [uneven, even, LC.tiny_volonex])
+@pytest.mark.parametrize("make", [uneven, bare, even, LC.tiny_volonex])
 def test_whole_prompt_layers_and_logits(make, dtype):
     M = Model(make(), dtype)
     for n in (1, 2, 23, 150):
@@ -441,7 +448,7 @@ def test_whole_prompt_layers_and_logits(make, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("make", [uneven, even])
+@pytest.mark.parametrize("make", [uneven, bare, even])
 def test_cuts_do_not_matter(make, dtype):
     """whole prompt = token by token = portions of changing size, down to two tokens, started anywhere in a chunk"""
     M = Model(make(), dtype)
