@@ -144,6 +144,27 @@ def kernels(size, batch=32, ctx=1024, prompt_seqs=4, prompt=2048):
             put("w8a8 " + name, phase, per_launch(lambda l: L.w8a8_gemm(xq, sx, wq[l], sw), len(wq)), N * K + M * K + M * N * 2, 2.0 * M * N * K, INT8_OPS)
             del wq
             torch.cuda.empty_cache()
+    # head, sampling and embedding rows
+    head = [D.DenseW(torch.randn((vocab, w), generator=gen, device="cuda", dtype=torch.bfloat16) * w ** -0.5, vocab, w) for _ in range(2)]
+    x = torch.randn((batch, w), generator=gen, device="cuda", dtype=torch.bfloat16)
+    put("volonex head (fp32 logits)", "decode", per_launch(lambda l: D.linear(x, head[l % 2], out_dtype=torch.float32), 4),
+        vocab * w * 2 + batch * (vocab * 4 + w * 2), 2.0 * batch * vocab * w, bf16)
+    lg = [torch.randn((batch, vocab), generator=gen, device="cuda") for _ in range(12)]
+    put("volonex argmax", "decode", per_launch(lambda l: A.argmax_rows(lg[l]), 12), batch * vocab * 4, 0.0, bf16)
+    lg = [v.to(torch.bfloat16) for v in lg + lg]
+    put("w8a8 argmax", "decode", per_launch(lambda l: A.argmax_rows(lg[l]), 24), batch * vocab * 2, 0.0, bf16)
+    wq = [torch.randint(-127, 128, (vocab, w), generator=gen, device="cuda", dtype=torch.int8) for _ in range(2)]
+    sw, sx = torch.full((vocab,), 0.01, device="cuda"), torch.full((batch,), 0.01, device="cuda")
+    xq = torch.randint(-127, 128, (batch, w), generator=gen, device="cuda", dtype=torch.int8)
+    put("w8a8 head", "decode", per_launch(lambda l: L.w8a8_gemm(xq, sx, wq[l % 2], sw), 4), vocab * w + batch * (vocab * 2 + w), 2.0 * batch * vocab * w, INT8_OPS)
+    Mp = prompt_seqs * prompt
+    ids = torch.randint(0, vocab, (Mp,), generator=gen, device="cuda")
+    st, h = D.rows(Mp, w, torch.float32, "cuda"), D.rows(Mp, w, torch.bfloat16, "cuda")
+    norm = D.DynamicTanh.of(0.5, torch.ones(w), torch.zeros(w), "cuda")
+    put("volonex embedding + norm", "prefill", per_launch(lambda l: D.embed_norm(ids, head[l % 2].data, w, 2.0, st, None, norm, h), 4), Mp * w * 8, 0.0, bf16)
+    put("w8a8 embedding", "prefill", per_launch(lambda l: A.embed_gather(ids, head[l % 2].data, out=h), 4), Mp * w * 4, 0.0, bf16)
+    del head, wq, lg, st, h
+    torch.cuda.empty_cache()
     # attention
     qkv_n = (H + 2 * G) * 128
     mp = (ctx + 127) // 128 * 128 // 16

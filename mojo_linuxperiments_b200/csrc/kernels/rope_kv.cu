@@ -155,6 +155,15 @@ __global__ void __launch_bounds__(256) argmax_rows_kernel(const T* logits, long 
       }
     }
     for (int i = c0 + nv * 8 + threadIdx.x; i < c1; i += blockDim.x) consider(logit_f(x[i]), i);
+  } else if (sizeof(T) == 4 && (reinterpret_cast<uintptr_t>(x + c0) & 15) == 0) {
+    const int nv = (c1 - c0) / 4;
+    const float4* xv = reinterpret_cast<const float4*>(x + c0);
+    for (int i = threadIdx.x; i < nv; i += blockDim.x) {
+      const float4 v = xv[i];
+      const int k = c0 + i * 4;
+      consider(v.x, k); consider(v.y, k + 1); consider(v.z, k + 2); consider(v.w, k + 3);
+    }
+    for (int i = c0 + nv * 4 + threadIdx.x; i < c1; i += blockDim.x) consider(logit_f(x[i]), i);
   } else {
     for (int i = c0 + threadIdx.x; i < c1; i += blockDim.x) consider(logit_f(x[i]), i);
   }
