@@ -26,7 +26,8 @@ NVCC_FLAGS = [
 ]
 # --use_fast_math is dropped for files whose numerics are compared bit-for-bit with an oracle
 # (act_quant) or that also carry the 32-bit form of a model
-NO_FAST_MATH = {"act_quant.cu", "bf16_gemm.cu", "bf16_gemm_decode.cu", "f32_gemm.cu", "rotary_paged.cu", "attn_paged.cu"}
+NO_FAST_MATH = {"act_quant.cu", "bf16_gemm.cu", "bf16_gemm_decode.cu", "f32_gemm.cu", "rotary_paged.cu", "attn_paged.cu", "latent.cu",
+                "mingru.cu", "moe_route.cu", "stream_rows.cu"}
 GXX_FLAGS = ["-O2", "-std=c++20", "-fPIC", "-Wall", "-Wextra", "-fno-stack-protector", "-pthread"]
 
 KERNEL_LIB = "libb200_kernels.so"
@@ -37,7 +38,8 @@ KERNEL_LIB = "libb200_kernels.so"
 # such model from a fresh checkout compiles.
 KERNEL_VARIANTS = {"": [], "trace": ["-DB200RT_TRACE"], "debug": ["-DB200RT_DEBUG"], "dense": []}
 KERNEL_SUBSETS = {"dense": ("attn_decode_paged.cu", "attn_paged.cu", "attn_prefill_paged.cu", "bf16_gemm.cu", "bf16_gemm_decode.cu",
-                            "f32_gemm.cu", "rope_kv.cu", "rotary_paged.cu", "tmap.cu", "trace.cu")}
+                            "f32_gemm.cu", "latent.cu", "mingru.cu", "moe.cu", "moe_route.cu", "rope_kv.cu", "rotary_paged.cu",
+                            "stream_rows.cu", "tmap.cu", "trace.cu")}
 
 
 HOSTRT_LIB = "libb200_hostrt.so"

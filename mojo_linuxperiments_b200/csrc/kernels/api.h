@@ -225,6 +225,7 @@ int b200_ep_combine_reduce(const int* ids_local, int M, int k, int d, int expert
 
 // ---- dense (unquantised) linears with a fused epilogue, dense_epilogue.cuh ---------------------------------------------
 enum { B200_EPI_STORE = 0, B200_EPI_RESIDUAL = 1, B200_EPI_GLU = 2 };
+enum { B200_ACT_NONE = 0, B200_ACT_RELU2 = 1 };                     // store: activation of the result (square of relu)
 typedef struct b200_dense_epilogue {
   int mode;
   int out_f32;                          // element type of y: 0 bf16, 1 fp32
@@ -235,7 +236,19 @@ typedef struct b200_dense_epilogue {
   float mult;                           // residual: factor on the linear's result
   const float* norm_w; const float* norm_b; float norm_alpha;     // dynamic tanh: tanh(alpha x) w + b
   float limit;                          // glu: bound of both branches
+  int act;                              // store: B200_ACT_*
+  const float* gate; long long ldg;     // store: gate logits [M][groups]: the result times their sigmoid, or NULL
+  long long y_group;                    // store: columns of y between groups
 } b200_dense_epilogue;
+// Several linears in one launch.  Their weights are stacked ([groups * N][K]); a group takes either all rows of x, at
+// columns g * x_group (heads), or the rows offsets[g] .. + counts[g] of x and y (experts).
+typedef struct b200_gemm_groups {
+  int groups;
+  long long x_group;
+  const int* offsets; const int* counts;               // NULL: every group takes all M rows
+  const void* tiles; const int* num_tiles; int max_tiles;      // int4 {group, first row, rows, 0} per 128 rows (prefill form)
+  int expected;                                        // about how many groups have rows (K split of the decode form); 0: all
+} b200_gemm_groups;
 // x [M][K] and w [N][K] with row pitches in elements (multiples of 8 for bf16, 16-byte aligned); force_bn 0 or 64 / 128 / 256.
 int b200_bf16_gemm(const void* x, long long ldx, const void* w, long long ldw, int M, int N, int K,
                    const b200_dense_epilogue* epi, int* status, int num_sms, int force_bn, cudaStream_t stream);
@@ -243,6 +256,45 @@ int b200_bf16_gemm_decode(const void* x, long long ldx, const void* w, long long
                           const b200_dense_epilogue* epi, int* status, int num_sms, int splits, cudaStream_t stream);
 int b200_f32_gemm(const float* x, long long ldx, const float* w, long long ldw, int M, int N, int K,
                   const b200_dense_epilogue* epi, cudaStream_t stream);
+
+// Grouped forms.  decode: M = most rows of a group, rows_total = rows of x.  prefill: row lists only.
+int b200_bf16_gemm_grouped(const void* x, long long ldx, const void* w, long long ldw, int rows_total, int N, int K,
+                           const b200_dense_epilogue* epi, const b200_gemm_groups* g, int* status, int num_sms, int force_bn,
+                           cudaStream_t stream);
+int b200_bf16_gemm_decode_grouped(const void* x, long long ldx, const void* w, long long ldw, int M, int rows_total, int N, int K,
+                                  const b200_dense_epilogue* epi, const b200_gemm_groups* g, int* status, int num_sms, int splits,
+                                  cudaStream_t stream);
+int b200_f32_gemm_grouped(const float* x, long long ldx, const float* w, long long ldw, int M, int N, int K,
+                          const b200_dense_epilogue* epi, const b200_gemm_groups* g, cudaStream_t stream);
+
+// ---- rows of the fp32 residual stream between two sub-layers whose norm needs the whole row (stream_rows.cu) ---------------
+// x' = source (+ mixture of experts) (+ add);  h = x' / rms(x') * gain;  with a token shift: h += (h of the previous token - h) * shift
+typedef struct b200_stream_rows {
+  const long long* ids; const void* table; long long ldt; int vocab, table_f32; float scale;    // source: embedding rows, or
+  const float* x; long long ldx; const long long* index;          // rows of the stream (row m is row index[m] if given)
+  const void* y; long long ldy; const int* slot; const int* chosen; const float* weight; int top, experts;   // expert results
+  const void* through; long long ldt2;                            // rows that experts numbered >= experts hand through
+  const float* add;                                               // [d], or NULL
+  float* x_out;                                                   // x' (pitch ldx, never x itself), or NULL
+  float gain, eps; void* h; long long ldh; int f32;               // element type of h, y and through
+  const float* shift; float* state; long long state_ld; int num_seqs;      // state: fp32 [num_seqs][state_ld], previous h
+  const int* positions; const int* seq_ids; const int* active;    // seq_ids NULL: row m is sequence m; active NULL: all
+  const int* cu; int portions, max_len;                           // shift: consecutive tokens; cu NULL: one token per portion
+} b200_stream_rows;
+int b200_stream_rows_launch(const b200_stream_rows* r, int M, int d, int num_sms, cudaStream_t stream);
+
+// ---- routing with a correction, expert groups and identity experts (moe_route.cu) ------------------------------------------
+int b200_route_grouped(const float* logits, long long ld, const float* correction, int M, int E, int top, int groups, int keep,
+                       float scale, int* ids, float* weights, cudaStream_t stream);
+int b200_moe_gather_rows(const void* x, long long row_bytes, const int* slot_token, const int* meta, int max_slots, void* out,
+                         cudaStream_t stream);
+
+// ---- gated linear recurrence over time (mingru.cu) ---------------------------------------------------------------------------
+// zxg fp32 [M][3 * width] (row pitch ld): S = (1 - sigmoid(z + zb)) S + sigmoid(z + zb) cand(x + xb); out = S silu(g).
+int b200_mingru_scratch_floats(int portions, int max_len, int width);
+int b200_mingru(const float* zxg, long long ld, const float* zb, const float* xb, int M, int width, float* state, long long state_ld,
+                int num_seqs, const int* positions, const int* seq_ids, const int* active, const int* cu, int portions, int max_len,
+                float* scratch, void* out, long long ldo, int f32, cudaStream_t stream);
 
 // ---- attention over a paged cache with free head sizes, optional chunk mask, sink and output gate ------------------------
 typedef struct b200_paged_cache {
@@ -278,6 +330,30 @@ int b200_attn_decode_paged(const void* qkv, long long ld, void* out, long long l
                            const int* seq_lens, const float* cos_tab, const float* sin_tab, int pairs, int interleaved,
                            int max_pos, const b200_paged_cache* cache, const b200_attn_spec* spec, int splits,
                            int* status, cudaStream_t stream);
+
+// ---- latent attention: the cache holds one normalised latent (rank) and one rotated key part (rot) per token ------------------
+// Cache descriptor: kv_heads 1, dk = rank + rot (each padded to 8), dv 0.
+typedef struct b200_latent_dims {
+  int heads, rank, rot;                 // padded to multiples of 8
+  int true_rank, true_rot;              // what the norm averages over, what turns
+} b200_latent_dims;
+// in fp32 [M][q_rank | rank | rot | ...]: norms of the query latent (-> cq) and of the latent, rotation of the key part;
+// the latter two go to the cache and, if given, to lat [M][rank + rot].
+int b200_latent_append(const float* in, long long ld, int M, int q_rank, int true_q_rank, const float* q_gain, const float* c_gain,
+                       float eps, const b200_latent_dims* dims, const int* positions, const int* seq_ids, const int* seq_lens,
+                       const float* cos_tab, const float* sin_tab, int max_pos, const b200_paged_cache* cache, void* cq,
+                       long long ldq, void* lat, int* status, cudaStream_t stream);
+// q [M][heads][head_ld]: pairs (2i, 2i+1) of the `true_rot` elements at `offset` of every head, in place
+int b200_rotary_heads(void* q, long long ld, int f32, int M, int heads, int head_ld, int offset, int true_rot, const int* positions,
+                      const float* cos_tab, const float* sin_tab, int max_pos, int* status, cudaStream_t stream);
+// cached rows 0 .. ctx[b+1] - ctx[b] of sequence seq_ids[b] -> lat [ctx[B]][dk]
+int b200_latent_gather(const b200_paged_cache* cache, const int* ctx, const int* seqs, int B, int max_ctx, void* lat, int* status,
+                       cudaStream_t stream);
+// General form, bf16 or fp32: q [M][heads][rank] against latents, q_rot [M][heads][rot] (already turned) against the key part;
+// out [M][heads][rank] = weighted latents.
+int b200_attn_latent_any(const void* q, long long ldq, const void* q_rot, long long ldr, int head_ld_rot, void* out, long long ldo,
+                         int M, const b200_latent_dims* dims, float scale, const int* positions, const int* seq_ids,
+                         const int* seq_lens, const b200_paged_cache* cache, int* status, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

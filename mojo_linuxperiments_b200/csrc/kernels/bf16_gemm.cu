@@ -10,6 +10,8 @@
 //   * Warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 epilogue.  An epilogue warp turns its 32 x 32 piece through
 //     shared memory, so that eight lanes share one token row and every global access is a run of 128 bytes: the residual
 //     form reads and writes fp32 rows.
+//   * Grouped form (experts): a table of row tiles names each tile's rows and its group, whose weights are rows
+//     group * N .. of one stacked matrix; a column tile that reaches into the next group's rows is cut in the epilogue.
 //   * Every wait is bounded; a CTA that gives up records a status code, drains and exits.
 #include "ptx.cuh"
 #include "api.h"
@@ -26,18 +28,29 @@ constexpr int BG_SP = 36;              // floats per row of an epilogue warp's s
 struct BfGemmParams {
   int M, N, m_tiles, n_tiles, kblocks, num_tiles;
   b200_dense_epilogue epi;
+  const int4* tiles; const int* tiles_used;      // row lists: {group, first row, rows, 0} per row tile, else NULL
   int* status;
   unsigned long long limit_ns;
 };
 
-__device__ __forceinline__ void bg_tile_coords(const BfGemmParams& p, int tile, int& m_tile, int& n_tile) {
+struct BfTile { int m0, m_end, n_tile, group; };
+
+__device__ __forceinline__ BfTile bg_tile_at(const BfGemmParams& p, int m_tiles, int tile) {
   const int per_group = BG_GROUP_M * p.n_tiles;
   const int g = tile / per_group;
   const int first_m = g * BG_GROUP_M;
-  const int gsize = min(BG_GROUP_M, p.m_tiles - first_m);
+  const int gsize = min(BG_GROUP_M, m_tiles - first_m);
   const int r = tile - g * per_group;
-  m_tile = first_m + r % gsize;
-  n_tile = r / gsize;
+  const int m_tile = first_m + r % gsize;
+  BfTile t;
+  t.n_tile = r / gsize;
+  if (p.tiles) {
+    const int4 e = p.tiles[m_tile];
+    t.group = e.x; t.m0 = e.y; t.m_end = e.y + e.z;
+  } else {
+    t.group = 0; t.m0 = m_tile * 128; t.m_end = p.M;
+  }
+  return t;
 }
 
 template <int BN, int STAGES>
@@ -79,6 +92,8 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
   const uint32_t tmem_base = *tmem_slot;
   const uint64_t limit = p.limit_ns;
   pdl_wait();                // everything before this kernel in the stream has completed
+  const int m_tiles = p.tiles ? min(*p.tiles_used, p.m_tiles) : p.m_tiles;
+  const int num_tiles = m_tiles * p.n_tiles;
 
   if (warp == 0) {
     if (lane == 0) {
@@ -87,15 +102,15 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
       const uint64_t pol_w = p.m_tiles == 1 ? policy_evict_first() : policy_evict_last();
       int stage = 0; uint32_t phase = 0;
       bool ok = true;
-      for (int tile = blockIdx.x; tile < p.num_tiles && ok; tile += gridDim.x) {
-        int m_tile, n_tile;
-        bg_tile_coords(p, tile, m_tile, n_tile);
+      for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
+        const BfTile t = bg_tile_at(p, m_tiles, tile);
+        const int w0 = t.group * p.N + t.n_tile * BN;
         for (int kb = 0; kb < p.kblocks; ++kb) {
           if (!mbar_wait(empty_bar(stage), phase ^ 1u, abort_flag, p.status, (ST_TIMEOUT_SMEM_EMPTY | (9 << 8)), limit)) { ok = false; break; }
           mbar_expect_tx(full_bar(stage), STAGE_BYTES);
           const uint32_t a_dst = smem_base + stage * STAGE_BYTES;
-          tma_load_2d(a_dst, &tmap_x, full_bar(stage), kb * 128, m_tile * 128);
-          tma_load_2d_hint(a_dst + A_BYTES, &tmap_w, full_bar(stage), kb * 128, n_tile * BN, pol_w);
+          tma_load_2d(a_dst, &tmap_x, full_bar(stage), kb * 128, t.m0);
+          tma_load_2d_hint(a_dst + A_BYTES, &tmap_w, full_bar(stage), kb * 128, w0, pol_w);
           if (++stage == STAGES) { stage = 0; phase ^= 1u; }
         }
       }
@@ -107,7 +122,7 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
       int stage = 0; uint32_t phase = 0;
       int idx = 0;
       bool ok = true;
-      for (int tile = blockIdx.x; tile < p.num_tiles && ok; tile += gridDim.x, ++idx) {
+      for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x, ++idx) {
         const int a = idx & 1;
         if (!mbar_wait(tempty_bar(a), ((idx >> 1) & 1u) ^ 1u, abort_flag, p.status, (ST_TIMEOUT_TMEM_EMPTY | (9 << 8)), limit)) { ok = false; break; }
         tc_fence_after();
@@ -132,11 +147,10 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
     int idx = 0;
     const bool residual = p.epi.mode == B200_EPI_RESIDUAL;
     const int rr0 = lane >> 3, c4 = (lane & 7) * 4;          // row group and column quad of this lane in a 32 x 32 piece
-    for (int tile = blockIdx.x; tile < p.num_tiles; tile += gridDim.x, ++idx) {
+    for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x, ++idx) {
       const int a = idx & 1;
-      int m_tile, n_tile;
-      bg_tile_coords(p, tile, m_tile, n_tile);
-      const int m0 = m_tile * 128 + q * 32, n0 = n_tile * BN;
+      const BfTile t = bg_tile_at(p, m_tiles, tile);
+      const int m0 = t.m0 + q * 32, n0 = t.n_tile * BN;
       // The residual rows of a piece are requested one piece ahead (the first even before the accumulator is complete):
       // the epilogue is four warps, so what it needs is loads in flight.
       float4 xn[8];
@@ -145,7 +159,7 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
 #pragma unroll
         for (int it = 0; it < 8; ++it) {
           const int m = m0 + it * 4 + rr0;
-          if (m < p.M && n < p.N) xn[it] = *reinterpret_cast<const float4*>(p.epi.x + static_cast<long long>(m) * p.epi.ldx + n);
+          if (m < t.m_end && n < p.N) xn[it] = *reinterpret_cast<const float4*>(p.epi.x + static_cast<long long>(m) * p.epi.ldx + n);
         }
       };
       if (residual) load_x(0);
@@ -179,13 +193,13 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
 #pragma unroll
             for (int it = 0; it < 8; ++it) {
               const int rr = it * 4 + rr0, m = m0 + rr;
-              if (m < p.M) epi_residual4(p.epi, nw, m, n, *reinterpret_cast<const float4*>(piece + rr * BG_SP + c4), xc[it]);
+              if (m < t.m_end) epi_residual4(p.epi, nw, m, n, *reinterpret_cast<const float4*>(piece + rr * BG_SP + c4), xc[it]);
             }
           } else {
 #pragma unroll
             for (int it = 0; it < 8; ++it) {
               const int rr = it * 4 + rr0, m = m0 + rr;
-              if (m < p.M) epi_apply4(p.epi, m, n, *reinterpret_cast<const float4*>(piece + rr * BG_SP + c4));
+              if (m < t.m_end) epi_apply4(p.epi, m, n, *reinterpret_cast<const float4*>(piece + rr * BG_SP + c4), t.group);
             }
           }
         }
@@ -233,20 +247,26 @@ int dense_epilogue_check(const b200_dense_epilogue* e, int N) {
 
 using namespace b200;
 
-extern "C" int b200_bf16_gemm(const void* x, long long ldx, const void* w, long long ldw, int M, int N, int K,
-                              const b200_dense_epilogue* epi, int* status, int num_sms, int force_bn, cudaStream_t stream) {
+// g NULL: one linear over M rows; else row lists over M = rows of x
+static int bf16_gemm_any(const void* x, long long ldx, const void* w, long long ldw, int M, int N, int K, const b200_dense_epilogue* epi,
+                         const b200_gemm_groups* g, int* status, int num_sms, int force_bn, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (N <= 0 || K <= 0 || ldx < K || ldw < K || (ldx % 8) || (ldw % 8)) return -1;
   if ((reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15)) return -2;
   if (int rc = dense_epilogue_check(epi, N)) return rc;
+  if (g && (g->groups <= 0 || !g->tiles || !g->num_tiles || g->max_tiles <= 0 || epi->mode != B200_EPI_STORE)) return -3;
   BfGemmParams p;
   p.M = M; p.N = N;
-  p.m_tiles = (M + 127) / 128;
+  p.m_tiles = g ? g->max_tiles : (M + 127) / 128;
+  p.tiles = g ? static_cast<const int4*>(g->tiles) : nullptr;
+  p.tiles_used = g ? g->num_tiles : nullptr;
+  // row lists: a partly filled tile per group on top of the full ones is what to expect
+  const int likely = g ? M / 128 + (g->expected > 0 ? g->expected : g->groups) : p.m_tiles;
   int bn = force_bn;
   if (bn != 64 && bn != 128 && bn != 256) {
     long long best_cost = -1;
     for (int cand : {256, 128, 64}) {
-      const long long tiles = static_cast<long long>(p.m_tiles) * ((N + cand - 1) / cand);
+      const long long tiles = static_cast<long long>(likely) * ((N + cand - 1) / cand);
       const long long cost = (tiles + num_sms - 1) / num_sms * (cand + 64);
       if (best_cost < 0 || cost < best_cost) { best_cost = cost; bn = cand; }
     }
@@ -259,11 +279,23 @@ extern "C" int b200_bf16_gemm(const void* x, long long ldx, const void* w, long 
   p.limit_ns = 2000000000ull;
   CUtensorMap tx, tw;
   if (make_tmap_2d_u8(&tx, x, static_cast<uint64_t>(K) * 2, M, static_cast<uint64_t>(ldx) * 2, 128)) return -11;
-  if (make_tmap_2d_u8(&tw, w, static_cast<uint64_t>(K) * 2, N, static_cast<uint64_t>(ldw) * 2, bn)) return -12;
+  if (make_tmap_2d_u8(&tw, w, static_cast<uint64_t>(K) * 2, static_cast<uint64_t>(N) * (g ? g->groups : 1), static_cast<uint64_t>(ldw) * 2, bn)) return -12;
   const int grid = p.num_tiles < num_sms ? p.num_tiles : num_sms;
   switch (bn) {
     case 64: return launch_bf16_gemm<64, 8>(tx, tw, p, grid, stream);
     case 128: return launch_bf16_gemm<128, 6>(tx, tw, p, grid, stream);
     default: return launch_bf16_gemm<256, 4>(tx, tw, p, grid, stream);
   }
+}
+
+extern "C" int b200_bf16_gemm(const void* x, long long ldx, const void* w, long long ldw, int M, int N, int K,
+                              const b200_dense_epilogue* epi, int* status, int num_sms, int force_bn, cudaStream_t stream) {
+  return bf16_gemm_any(x, ldx, w, ldw, M, N, K, epi, nullptr, status, num_sms, force_bn, stream);
+}
+
+extern "C" int b200_bf16_gemm_grouped(const void* x, long long ldx, const void* w, long long ldw, int rows_total, int N, int K,
+                                      const b200_dense_epilogue* epi, const b200_gemm_groups* g, int* status, int num_sms,
+                                      int force_bn, cudaStream_t stream) {
+  if (!g) return -3;
+  return bf16_gemm_any(x, ldx, w, ldw, rows_total, N, K, epi, g, status, num_sms, force_bn, stream);
 }

@@ -9,6 +9,9 @@
 //     to the owner as fp32 through distributed shared memory ([sender][token][channel]), the owner adds them in rank
 //     order (the result does not depend on timing) and runs the epilogue on four channels of a token at a time.
 //   * More than BN tokens: blockIdx.z picks the token block; the weights come from L2 the second time.
+//   * Grouped form: blockIdx.z also picks the group, whose weights are rows group * N .. of one stacked matrix (a tile that
+//     reaches into the next group's rows is cut in the epilogue).  Heads take all rows at their own columns of x; experts
+//     take their own rows, known only once the routing kernel has finished, so those CTAs wait first and leave if idle.
 #include "ptx.cuh"
 #include "api.h"
 #include "launch.cuh"
@@ -21,6 +24,9 @@ int dense_epilogue_check(const b200_dense_epilogue* e, int N);
 
 struct BfDecodeParams {
   int M, N, kblocks, splits;
+  int z_tiles, groups;                  // groups 0: one linear
+  int x_group_bytes;
+  const int* offsets; const int* counts;
   b200_dense_epilogue epi;
   int* status;
   unsigned long long limit_ns;
@@ -59,7 +65,16 @@ bf16_gemm_decode_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid
 
   const int S = p.splits;
   const int rank = static_cast<int>(cluster_ctarank());
-  const int n_tile = blockIdx.y, m0 = blockIdx.z * BN, rows = min(BN, p.M - m0);
+  const int grp = p.groups > 0 ? blockIdx.z / p.z_tiles : 0, zt = blockIdx.z - grp * p.z_tiles;
+  const int n_tile = blockIdx.y;
+  int m0 = zt * BN, rows = min(BN, p.M - m0);
+  if (p.counts) {
+    pdl_wait();
+    rows = min(BN, p.counts[grp] - m0);
+    if (rows <= 0) return;                      // the whole cluster
+    m0 += p.offsets[grp];
+  }
+  const int w0 = grp * p.N + n_tile * 128, x0 = grp * p.x_group_bytes;
   const int kb0 = static_cast<int>(static_cast<long long>(p.kblocks) * rank / S);
   const int kb1 = static_cast<int>(static_cast<long long>(p.kblocks) * (rank + 1) / S);
   const uint64_t limit = p.limit_ns;
@@ -85,10 +100,10 @@ bf16_gemm_decode_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid
       const int pre = min(STAGES, kb1 - kb0);
       for (int i = 0; i < pre; ++i) {
         mbar_expect_tx(full_bar(i), STAGE_BYTES);
-        tma_load_2d_hint(smem_base + i * STAGE_BYTES, &tmap_w, full_bar(i), (kb0 + i) * 128, n_tile * 128, pol_w);
+        tma_load_2d_hint(smem_base + i * STAGE_BYTES, &tmap_w, full_bar(i), (kb0 + i) * 128, w0, pol_w);
       }
       pdl_wait();
-      for (int i = 0; i < pre; ++i) tma_load_2d(smem_base + i * STAGE_BYTES + A_BYTES, &tmap_x, full_bar(i), (kb0 + i) * 128, m0);
+      for (int i = 0; i < pre; ++i) tma_load_2d(smem_base + i * STAGE_BYTES + A_BYTES, &tmap_x, full_bar(i), x0 + (kb0 + i) * 128, m0);
       bool ok = true;
       int stage = pre == STAGES ? 0 : pre;
       uint32_t phase = pre == STAGES ? 1u : 0u;
@@ -96,8 +111,8 @@ bf16_gemm_decode_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid
         if (!mbar_wait(empty_bar(stage), phase ^ 1u, abort_flag, p.status, (ST_TIMEOUT_SMEM_EMPTY | (10 << 8)), limit)) { ok = false; break; }
         mbar_expect_tx(full_bar(stage), STAGE_BYTES);
         const uint32_t a_dst = smem_base + stage * STAGE_BYTES;
-        tma_load_2d_hint(a_dst, &tmap_w, full_bar(stage), kb * 128, n_tile * 128, pol_w);
-        tma_load_2d(a_dst + A_BYTES, &tmap_x, full_bar(stage), kb * 128, m0);
+        tma_load_2d_hint(a_dst, &tmap_w, full_bar(stage), kb * 128, w0, pol_w);
+        tma_load_2d(a_dst + A_BYTES, &tmap_x, full_bar(stage), x0 + kb * 128, m0);
         if (++stage == STAGES) { stage = 0; phase ^= 1u; }
       }
       if (!ok) { const uint64_t t0 = globaltimer_ns(); while (globaltimer_ns() - t0 < 2000000ull) { } }   // copies in flight land
@@ -166,7 +181,7 @@ bf16_gemm_decode_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid
       const float4 u = *reinterpret_cast<const float4*>(ex + (s * BN + j) * cwp + c4);
       v.x += u.x; v.y += u.y; v.z += u.z; v.w += u.w;
     }
-    epi_apply4(p.epi, m0 + j, n, v);
+    epi_apply4(p.epi, m0 + j, n, v, grp);
   }
 
   __syncthreads();
@@ -203,38 +218,63 @@ static int bd_resident(int S, int num_sms, int per_sm) {
 
 using namespace b200;
 
-// At most 128 tokens.  splits: 0 picks the K split, else 1..8 CTAs per cluster.
-extern "C" int b200_bf16_gemm_decode(const void* x, long long ldx, const void* w, long long ldw, int M, int N, int K,
-                                     const b200_dense_epilogue* epi, int* status, int num_sms, int splits, cudaStream_t stream) {
-  if (M <= 0) return 0;
-  if (M > 128 || N <= 0 || K <= 0 || ldx < K || ldw < K || (ldx % 8) || (ldw % 8) || splits < 0 || splits > 8) return -1;
+// splits: 0 picks the K split, else 1..8 CTAs per cluster
+static int bf16_decode_any(const void* x, long long ldx, const void* w, long long ldw, int M, int rows_total, int N, int K,
+                           const b200_dense_epilogue* epi, const b200_gemm_groups* g, int* status, int num_sms, int splits, cudaStream_t stream) {
+  if (M <= 0 || rows_total <= 0) return 0;
+  if (N <= 0 || K <= 0 || ldx < K || ldw < K || (ldx % 8) || (ldw % 8) || splits < 0 || splits > 8) return -1;
   if ((reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15)) return -2;
   if (int rc = dense_epilogue_check(epi, N)) return rc;
-  const int bn = M <= 16 ? 16 : (M <= 32 ? 32 : 64);
+  if (g && (g->groups <= 0 || g->x_group % 8 || g->x_group < 0 || (g->counts && !g->offsets) || epi->mode != B200_EPI_STORE)) return -3;
+  const bool lists = g && g->counts;
+  if (g && !lists && (g->groups - 1) * g->x_group + K > ldx) return -3;
+  const int bn = lists || M <= 16 ? 16 : (M <= 32 ? 32 : 64);
   BfDecodeParams p;
   p.M = M; p.N = N;
   p.kblocks = (K + 63) / 64;
+  p.z_tiles = (M + bn - 1) / bn;
+  p.groups = g ? g->groups : 0;
+  p.x_group_bytes = g && !lists ? static_cast<int>(g->x_group * 2) : 0;
+  p.offsets = lists ? g->offsets : nullptr;
+  p.counts = lists ? g->counts : nullptr;
   p.epi = *epi;
   p.status = status;
   p.limit_ns = 2000000000ull;
-  const int n_tiles = (N + 127) / 128, z = (M + bn - 1) / bn;
+  const int n_tiles = (N + 127) / 128, z = p.z_tiles * (g ? g->groups : 1);
+  if (z > 65535) return -4;
   if (splits == 0) {
     double best = 0;
+    const int busy = lists && g->expected > 0 && g->expected < g->groups ? g->expected : (lists ? g->groups : z);
     for (int s = 1; s <= 8 && s <= p.kblocks; ++s) {
-      const int clusters = n_tiles * z, res = bd_resident(s, num_sms, bn == 64 ? 1 : 2);
+      const int clusters = n_tiles * busy, res = bd_resident(s, num_sms, bn == 64 ? 1 : 2);
       const double cost = static_cast<double>((clusters + res - 1) / res) * ((p.kblocks + s - 1) / s + 6 + (s > 1 ? 1 : 0));
       if (splits == 0 || cost < best) { best = cost; splits = s; }
     }
   }
   if (splits > p.kblocks) splits = p.kblocks;
   p.splits = splits;
+  const uint64_t x_cols = static_cast<uint64_t>(g && !lists ? (g->groups - 1) * g->x_group + K : K);
   CUtensorMap tw, tx;
-  if (make_tmap_2d_u8(&tw, w, static_cast<uint64_t>(K) * 2, N, static_cast<uint64_t>(ldw) * 2, 128)) return -11;
-  if (make_tmap_2d_u8(&tx, x, static_cast<uint64_t>(K) * 2, M, static_cast<uint64_t>(ldx) * 2, bn)) return -12;
+  if (make_tmap_2d_u8(&tw, w, static_cast<uint64_t>(K) * 2, static_cast<uint64_t>(N) * (g ? g->groups : 1), static_cast<uint64_t>(ldw) * 2, 128)) return -11;
+  if (make_tmap_2d_u8(&tx, x, x_cols * 2, rows_total, static_cast<uint64_t>(ldx) * 2, bn)) return -12;
   const dim3 grid(splits, n_tiles, z);
   switch (bn) {
     case 16: return launch_bf16_decode<16, 5>(tw, tx, p, grid, stream);
     case 32: return launch_bf16_decode<32, 4>(tw, tx, p, grid, stream);
     default: return launch_bf16_decode<64, 6>(tw, tx, p, grid, stream);
   }
+}
+
+// At most 128 tokens.
+extern "C" int b200_bf16_gemm_decode(const void* x, long long ldx, const void* w, long long ldw, int M, int N, int K,
+                                     const b200_dense_epilogue* epi, int* status, int num_sms, int splits, cudaStream_t stream) {
+  if (M > 128) return -1;
+  return bf16_decode_any(x, ldx, w, ldw, M, M, N, K, epi, nullptr, status, num_sms, splits, stream);
+}
+
+extern "C" int b200_bf16_gemm_decode_grouped(const void* x, long long ldx, const void* w, long long ldw, int M, int rows_total, int N,
+                                             int K, const b200_dense_epilogue* epi, const b200_gemm_groups* g, int* status,
+                                             int num_sms, int splits, cudaStream_t stream) {
+  if (!g) return -3;
+  return bf16_decode_any(x, ldx, w, ldw, M, rows_total, N, K, epi, g, status, num_sms, splits, stream);
 }

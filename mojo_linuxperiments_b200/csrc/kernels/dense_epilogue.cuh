@@ -1,6 +1,7 @@
 // What happens to a finished value of a dense (unquantised) linear before it leaves the kernel.
 //
-//   store     y[m][n] = v
+//   store     y[m][n] = v, optionally after an activation (square of relu) and times the sigmoid of a gate per (row, group);
+//             grouped linears put group g at column g * y_group
 //   residual  x[m][n] += mult * v (fp32, in place), optionally + add[m][n]; then, if y is given, the norm of the *next*
 //             sub-layer is applied to the new residual and y[m][n] = norm(x) - possible here because the norm is
 //             element-wise (dynamic tanh), so no second pass over the row is needed
@@ -72,11 +73,19 @@ __device__ __forceinline__ void epi_residual4(const b200_dense_epilogue& e, cons
   if (e.y) store4_any(e.y, e.out_f32 != 0, m * e.ldy + n, epi_norm4(e, k, x, e.exact != 0));
 }
 
-// columns n .. n+3 (n a multiple of four, n < N) of row m
-__device__ __forceinline__ void epi_apply4(const b200_dense_epilogue& e, long long m, int n, float4 v) {
+// columns n .. n+3 (n a multiple of four, n < N) of row m of group g
+__device__ __forceinline__ void epi_apply4(const b200_dense_epilogue& e, long long m, int n, float4 v, int g = 0) {
   const bool f32 = e.out_f32 != 0;
   if (e.mode == B200_EPI_STORE) {
-    store4_any(e.y, f32, m * e.ldy + n, v);
+    if (e.act == B200_ACT_RELU2) {
+      v.x = fmaxf(v.x, 0.f); v.y = fmaxf(v.y, 0.f); v.z = fmaxf(v.z, 0.f); v.w = fmaxf(v.w, 0.f);
+      v.x *= v.x; v.y *= v.y; v.z *= v.z; v.w *= v.w;
+    }
+    if (e.gate) {
+      const float s = epi_sigmoid(e.gate[m * e.ldg + g], e.exact != 0);
+      v.x *= s; v.y *= s; v.z *= s; v.w *= s;
+    }
+    store4_any(e.y, f32, m * e.ldy + g * e.y_group + n, v);
   } else if (e.mode == B200_EPI_GLU) {
     const bool exact = e.exact != 0;
     const float g0 = fminf(v.x, e.limit), u0 = fminf(fmaxf(v.y, -e.limit), e.limit);

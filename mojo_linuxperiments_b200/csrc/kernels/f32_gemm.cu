@@ -14,9 +14,17 @@ constexpr int FG_T = 64, FG_K = 16, FG_P = FG_T + 4;
 
 __global__ void __launch_bounds__(256)
 f32_gemm_kernel(const float* x, long long ldx, const float* w, long long ldw, int M, int N, int K,
-                const __grid_constant__ b200_dense_epilogue epi) {
+                const __grid_constant__ b200_dense_epilogue epi, const __grid_constant__ b200_gemm_groups gr) {
   pdl_launch_dependents();
   pdl_wait();
+  const int grp = blockIdx.z;
+  int base = 0;                                      // first row of this group
+  if (gr.groups > 0) {
+    w += static_cast<long long>(grp) * N * ldw;
+    if (gr.counts) { base = gr.offsets[grp]; M = min(M, gr.counts[grp]); x += base * ldx; }
+    else x += grp * gr.x_group;
+    if (static_cast<int>(blockIdx.y) * FG_T >= M) return;
+  }
   __shared__ __align__(16) float xs[FG_K][FG_P], ws[FG_K][FG_P];
   const int m0 = blockIdx.y * FG_T, n0 = blockIdx.x * FG_T;
   const int lr = threadIdx.x >> 2, lk = (threadIdx.x & 3) * 4;      // loader: one row, four consecutive k
@@ -49,7 +57,7 @@ f32_gemm_kernel(const float* x, long long ldx, const float* w, long long ldw, in
   if (n0 + tn < N) {
 #pragma unroll
     for (int i = 0; i < 4; ++i)
-      if (m0 + tm + i < M) epi_apply4(epi, m0 + tm + i, n0 + tn, make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]));
+      if (m0 + tm + i < M) epi_apply4(epi, base + m0 + tm + i, n0 + tn, make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]), grp);
   }
 }
 
@@ -57,12 +65,20 @@ f32_gemm_kernel(const float* x, long long ldx, const float* w, long long ldw, in
 
 using namespace b200;
 
-extern "C" int b200_f32_gemm(const float* x, long long ldx, const float* w, long long ldw, int M, int N, int K,
-                             const b200_dense_epilogue* epi, cudaStream_t stream) {
+extern "C" int b200_f32_gemm_grouped(const float* x, long long ldx, const float* w, long long ldw, int M, int N, int K,
+                                     const b200_dense_epilogue* epi, const b200_gemm_groups* g, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (N <= 0 || K <= 0 || ldx < K || ldw < K || (M + FG_T - 1) / FG_T > 65535) return -1;
+  b200_gemm_groups none = {};
+  if (g && (g->groups <= 0 || g->groups > 65535 || (g->counts && !g->offsets) || !epi || epi->mode != B200_EPI_STORE)) return -1;
   if (int rc = dense_epilogue_check(epi, N)) return rc;
-  launch_ex(f32_gemm_kernel, dim3((N + FG_T - 1) / FG_T, (M + FG_T - 1) / FG_T), dim3(256), 0, stream, 0, x, ldx, w, ldw, M, N, K, *epi);
+  launch_ex(f32_gemm_kernel, dim3((N + FG_T - 1) / FG_T, (M + FG_T - 1) / FG_T, g ? g->groups : 1), dim3(256), 0, stream, 0,
+            x, ldx, w, ldw, M, N, K, *epi, g ? *g : none);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -2000 - static_cast<int>(e);
+}
+
+extern "C" int b200_f32_gemm(const float* x, long long ldx, const float* w, long long ldw, int M, int N, int K,
+                             const b200_dense_epilogue* epi, cudaStream_t stream) {
+  return b200_f32_gemm_grouped(x, ldx, w, ldw, M, N, K, epi, nullptr, stream);
 }

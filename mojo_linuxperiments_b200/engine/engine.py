@@ -79,7 +79,7 @@ class Engine:
             self.kv = KVState(self.cfg, self.rt, self.device, batch, self.rt.max_seq_len, alloc=self.runtime.zeros)
             self.tokens = torch.zeros(batch, dtype=torch.int64, device=self.device)
             self.positions = torch.zeros(batch, dtype=torch.int32, device=self.device)
-            self.active = torch.zeros(batch, dtype=torch.int32, device=self.device)
+            self.active = self.kv.active        # kernels that carry a state from token to token read it
         else:
             # same cache, same static tensors: the captured graphs stay valid
             for s in list(self.kv.owned):
@@ -308,10 +308,11 @@ class Engine:
                     room -= n
             if not part:
                 break
-            ids, pos, sid, cu, rows, got = [], [], [], [0], [], []
+            ids, pos, sid, cu, rows, got, starts = [], [], [], [0], [], [], []
             for i, a, n in part:
                 slot, toks, want = entries[i]
                 start = self._lens[slot]
+                starts.append(start)
                 self.kv.retire(slot, start)
                 self.kv.admit(slot, start + n)
                 ids.append(toks[a:a + n])
@@ -329,7 +330,8 @@ class Engine:
             nxt = self.model.forward(torch.cat(ids).to(dev, non_blocking=True), torch.cat(pos).to(dev, non_blocking=True), self.kv,
                                      mode="prefill", cu_seqlens=torch.tensor(cu, dtype=torch.int32).to(dev, non_blocking=True),
                                      max_len=max(n for _, _, n in part), seq_ids=torch.cat(sid).to(dev, non_blocking=True),
-                                     last_idx=last.to(dev, non_blocking=True))
+                                     last_idx=last.to(dev, non_blocking=True),
+                                     portions=[(a, n) for a, (_, _, n) in zip(starts, part)])
             default_workspace(dev).next_step()
             for i, ks, r0, final in got:
                 out[i].index_copy_(0, torch.tensor(ks, dtype=torch.int64).to(dev, non_blocking=True),
@@ -443,14 +445,15 @@ class Engine:
         g = self._graphs.get(self.batch)
         if g is None:
             # warm up outside capture (lazy kernel attribute set-up, allocator), restoring the state afterwards
-            saved = (self.tokens.clone(), self.positions.clone(), self.kv.seq_lens.clone())
+            saved = (self.tokens.clone(), self.positions.clone(), self.kv.seq_lens.clone(), self.active.clone())
+            self.active.zero_()         # the rehearsal must not move the sequences' states on
             self._stream.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(self._stream):
                 self._decode_body()
             torch.cuda.current_stream().wait_stream(self._stream)
             torch.cuda.synchronize()
             self.check_status()         # a bounded wait that ran out surfaces here, before anything is captured or timed
-            self.tokens.copy_(saved[0]); self.positions.copy_(saved[1]); self.kv.seq_lens.copy_(saved[2])
+            self.tokens.copy_(saved[0]); self.positions.copy_(saved[1]); self.kv.seq_lens.copy_(saved[2]); self.active.copy_(saved[3])
             g = torch.cuda.CUDAGraph()
             from ..ops import _lib
             n0 = _lib.LAUNCHES[0]

@@ -16,7 +16,7 @@ class CacheSpec:
     """What one layer (one pass of it, if layers repeat) keeps per token in the paged cache."""
     kv_heads: int
     dk: int                       # stored key size per head
-    dv: int                       # stored value size per head
+    dv: int                       # stored value size per head; 0: the values are computed from the keys (latents)
     dtype: str = "bfloat16"
     chunk: int | None = None      # positions only see their own block of this many positions; None: all earlier ones
 

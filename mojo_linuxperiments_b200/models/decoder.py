@@ -144,7 +144,7 @@ class Decoder:
     # -- full forward ------------------------------------------------------------------------------------------
     def forward(self, token_ids: torch.Tensor, positions: torch.Tensor, kv: KVState, *, mode: str,
                 cu_seqlens: torch.Tensor | None = None, max_len: int = 0, seq_ids: torch.Tensor | None = None,
-                last_idx: torch.Tensor | None = None) -> torch.Tensor:
+                last_idx: torch.Tensor | None = None, portions: list | None = None) -> torch.Tensor:
         """token_ids int64 [M], positions int32 [M] -> greedy next token per sequence (int64).
 
         mode "prefill": M = all prompt tokens (concatenated), ``last_idx`` selects each sequence's last row;

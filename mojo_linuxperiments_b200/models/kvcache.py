@@ -3,7 +3,11 @@
 Every model family describes what its layers store (``cfg.cache_layout``: heads, key and value sizes, element type, how
 far back a position looks); pages of 16 tokens (``rt.page_size``) are handed out per sequence and shared by all layers,
 i.e. page *p* of a sequence is record *p* of every layer's storage.  Layers that look back only to the start of their
-own chunk let go of older tokens: when no layer can see a page any more it returns to the free list (``retire``)."""
+own chunk let go of older tokens: when no layer can see a page any more it returns to the free list (``retire``).
+
+Beside the pages every sequence slot has a fixed-size fp32 state per layer (``cfg.state_layout``: the previous token's row
+of a token shift, the state of a recurrence).  Kernels take a sequence's state as zero at position 0, so a slot needs no
+clearing between sequences, and change it only where ``active`` says that the slot takes part in the step."""
 from __future__ import annotations
 
 import torch
@@ -14,8 +18,12 @@ from .config import CacheSpec, ModelConfig, RuntimeConfig
 _DTYPES = {"bfloat16": torch.bfloat16, "float32": torch.float32}
 
 
-def _record(s: CacheSpec, page_size: int) -> int:
-    return s.kv_heads * page_size * (s.dk + s.dv)
+def _record(s: CacheSpec | None, page_size: int) -> int:
+    return s.kv_heads * page_size * (s.dk + s.dv) if s is not None else 0
+
+
+def _states(cfg) -> list[dict[str, int]]:
+    return cfg.state_layout() if hasattr(cfg, "state_layout") else []
 
 
 class KVState:
@@ -24,10 +32,10 @@ class KVState:
         """Pages the free list starts with: what the slots can hold at once, unless ``rt.kv_pool_tokens`` says less."""
         ps = rt.page_size
         per_seq = (max_seq_len + ps - 1) // ps
-        chunks = [s.chunk for s in cfg.cache_layout(rt)]
+        chunks = [s.chunk for s in cfg.cache_layout(rt) if s is not None]
         if all(chunks):
             # what lies before the oldest visible chunk is given back between portions of a prompt
-            per_seq = min(per_seq, (max(chunks) + rt.max_prefill_tokens + ps - 1) // ps + 2)
+            per_seq = min(per_seq, (max(chunks, default=0) + rt.max_prefill_tokens + ps - 1) // ps + 2)
         total = num_seqs * per_seq
         if rt.kv_pool_tokens > 0:
             total = min(total, (rt.kv_pool_tokens + ps - 1) // ps + 2 * num_seqs)
@@ -39,8 +47,10 @@ class KVState:
         max_pages = (max_seq_len + rt.page_size - 1) // rt.page_size
         pages = KVState.pool_pages(cfg, rt, num_seqs, max_seq_len) + 1
         layout = cfg.cache_layout(rt)
-        size = _DTYPES[layout[0].dtype].itemsize
-        return sum(_record(s, rt.page_size) for s in layout) * pages * size + num_seqs * max_pages * 4 + num_seqs * 4 + 3 * 1024
+        size = max((_DTYPES[s.dtype].itemsize for s in layout if s is not None), default=0)
+        states = sum(n for run in _states(cfg) for n in run.values()) * num_seqs * 4
+        return (sum(_record(s, rt.page_size) for s in layout) * pages * size + states + num_seqs * max_pages * 4 + num_seqs * 8 +
+                5 * 1024 + 512 * len(layout))
 
     def __init__(self, cfg: ModelConfig, rt: RuntimeConfig, device, num_seqs: int, max_seq_len: int, alloc=None):
         """``alloc(shape, dtype) -> zeroed tensor``: where the cache lives (the rank's HBM arena); default torch.zeros.
@@ -57,14 +67,25 @@ class KVState:
         self.num_pages = self.pool_pages(cfg, rt, num_seqs, max_seq_len) + 1
         self.scratch_page = self.num_pages - 1
         self.layout = cfg.cache_layout(rt)
-        assert len({s.dtype for s in self.layout}) == 1
+        assert len({s.dtype for s in self.layout if s is not None}) <= 1
         sizes = [_record(s, rt.page_size) * self.num_pages for s in self.layout]
-        self.storage = alloc((sum(sizes),), _DTYPES[self.layout[0].dtype])
+        dtype = next((s.dtype for s in self.layout if s is not None), rt.dtype)
+        self.storage = alloc((max(1, sum(sizes)),), _DTYPES[dtype])
         self.layers, at = [], 0
         for s, n in zip(self.layout, sizes):
             self.layers.append(A.PagedKVCache(self.num_pages, s.kv_heads, rt.page_size, device, storage=self.storage[at:at + n],
-                                              dk=s.dk, dv=s.dv))
+                                              dk=s.dk, dv=s.dv) if s is not None else None)
             at += n
+        # [sequence][numbers] per run and name; the numbers of a run are multiples of eight
+        self.states: list[dict[str, torch.Tensor]] = []
+        layout = _states(cfg)
+        flat, at = alloc((max(1, sum(n for run in layout for n in run.values()) * num_seqs),), torch.float32), 0
+        for run in layout:
+            self.states.append({})
+            for name, n in run.items():
+                self.states[-1][name] = flat[at:at + n * num_seqs].view(num_seqs, n)
+                at += n * num_seqs
+        self.active = alloc((num_seqs,), torch.int32)         # 1: the slot takes part in the next decode step
         self.page_table = alloc((num_seqs, self.max_pages), torch.int32)
         self.seq_lens = alloc((num_seqs,), torch.int32)
         self.free_pages = list(range(self.num_pages - 2, -1, -1))
@@ -95,7 +116,7 @@ class KVState:
 
     def first_visible(self, pos: int) -> int:
         """Oldest position that some layer of a token at ``pos`` (or any later one) can still see."""
-        return min((pos - pos % s.chunk) if s.chunk else 0 for s in self.layout)
+        return min(((pos - pos % s.chunk) if s.chunk else 0 for s in self.layout if s is not None), default=pos)
 
     def retire(self, seq: int, pos: int) -> None:
         """The next token of slot ``seq`` goes to position ``pos``: pages that lie wholly before everything it can see

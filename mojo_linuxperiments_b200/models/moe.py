@@ -14,8 +14,10 @@ from __future__ import annotations
 
 import torch
 
+from ..ops import dense as D
 from ..ops import linear as L
 from ..ops import moe as MO
+from ..ops import rows as RW
 
 
 class MoEBlock:
@@ -54,3 +56,20 @@ class MoEBlock:
         hq, sh = L.act_quant(gu, mode=L.AQ_SWIGLU)
         yd = MO.grouped_gemm(hq, sh, W["experts_down"].qweight, W["experts_down"].scale, work)
         return sp.ep_combine(yd, work, wts, ids_loc, M, self.n_local)
+
+
+class GroupedExperts:
+    """Mixture of ungated bf16 / fp32 experts on one GPU: routing with a correction and expert groups, grouped linears with the
+    squared-relu activation in the epilogue; the weighted sum is left to whoever reads the rows next (``ExpertSum``)."""
+
+    def __init__(self, spec):
+        self.m = spec
+
+    def __call__(self, h: torch.Tensor, W: dict) -> RW.ExpertSum:
+        m = self.m
+        logits = D.linear(h, W["router"], out_dtype=torch.float32)
+        ids, wts = MO.route_grouped(logits, W["correction"], m.top, m.groups, m.keep, m.scale, m.outputs)
+        work = MO.moe_align(ids, 0, m.experts)
+        u = D.linear_experts(MO.gather_rows(h, work), W["experts_up"], work, act="relu2")
+        y = D.linear_experts(u, W["experts_down"], work)
+        return RW.ExpertSum(y, work.inv, ids, wts, m.experts, h)

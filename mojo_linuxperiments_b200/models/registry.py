@@ -40,8 +40,9 @@ def _layered() -> Family:
                   lambda path, rt, rank, device: LW.load(path, rt, device))
 
 
-ARCHITECTURES = {"Volonex": _layered}       # config.json "architecture" -> family
-PRESETS = {**W8A8_PRESETS, "volonex-8b": LC.volonex_8b, "volonex-1b": LC.volonex_1b, "tiny-volonex": LC.tiny_volonex}
+ARCHITECTURES = {name: _layered for name in LC.DESIGNS}       # config.json "architecture" -> family
+PRESETS = {**W8A8_PRESETS, "volonex-8b": LC.volonex_8b, "volonex-1b": LC.volonex_1b, "tiny-volonex": LC.tiny_volonex,
+           "rakelorn-16b": LC.rakelorn_16b, "rakelorn-2b": LC.rakelorn_2b, "tiny-rakelorn": LC.tiny_rakelorn}
 
 
 def family_of(cfg) -> Family:

@@ -101,6 +101,18 @@ class _Sig:
     b200_bf16_gemm = (I, [P, LL, P, LL, I, I, I, P, P, I, I, P])
     b200_bf16_gemm_decode = (I, [P, LL, P, LL, I, I, I, P, P, I, I, P])
     b200_f32_gemm = (I, [P, LL, P, LL, I, I, I, P, P])
+    b200_bf16_gemm_grouped = (I, [P, LL, P, LL, I, I, I, P, P, P, I, I, P])
+    b200_bf16_gemm_decode_grouped = (I, [P, LL, P, LL, I, I, I, I, P, P, P, I, I, P])
+    b200_f32_gemm_grouped = (I, [P, LL, P, LL, I, I, I, P, P, P])
+    b200_stream_rows_launch = (I, [P, I, I, I, P])
+    b200_route_grouped = (I, [P, LL, P, I, I, I, I, I, F, P, P, P])
+    b200_moe_gather_rows = (I, [P, LL, P, P, I, P, P])
+    b200_mingru_scratch_floats = (I, [I, I, I])
+    b200_mingru = (I, [P, LL, P, P, I, I, P, LL, I, P, P, P, P, I, I, P, P, LL, I, P])
+    b200_latent_append = (I, [P, LL, I, I, I, P, P, F, P, P, P, P, P, P, I, P, P, LL, P, P, P])
+    b200_rotary_heads = (I, [P, LL, I, I, I, I, I, I, P, P, P, I, P, P])
+    b200_latent_gather = (I, [P, P, P, I, I, P, P, P])
+    b200_attn_latent_any = (I, [P, LL, P, LL, I, P, LL, I, P, F, P, P, P, P, P, P])
     b200_rotary_paged = (I, [P, LL, I, I, P, P, P, P, I, I, I, P, P, P])
     b200_embed_norm = (I, [P, P, LL, I, I, F, I, I, P, P, P, P])
     b200_attn_paged = (I, [P, LL, P, LL, I, I, P, P, P, P, P, P, P])
@@ -131,7 +143,30 @@ class DenseEpilogue(ctypes.Structure):
     """``b200_dense_epilogue`` of csrc/kernels/api.h: what a dense linear does with its result."""
     _fields_ = [("mode", c_int), ("out_f32", c_int), ("exact", c_int), ("y", c_void_p), ("ldy", c_longlong), ("x", c_void_p),
                 ("ldx", c_longlong), ("add", c_void_p), ("mult", c_float), ("norm_w", c_void_p), ("norm_b", c_void_p),
-                ("norm_alpha", c_float), ("limit", c_float)]
+                ("norm_alpha", c_float), ("limit", c_float), ("act", c_int), ("gate", c_void_p), ("ldg", c_longlong),
+                ("y_group", c_longlong)]
+
+
+class GemmGroups(ctypes.Structure):
+    """``b200_gemm_groups`` of csrc/kernels/api.h: several linears in one launch."""
+    _fields_ = [("groups", c_int), ("x_group", c_longlong), ("offsets", c_void_p), ("counts", c_void_p), ("tiles", c_void_p),
+                ("num_tiles", c_void_p), ("max_tiles", c_int), ("expected", c_int)]
+
+
+class StreamRows(ctypes.Structure):
+    """``b200_stream_rows`` of csrc/kernels/api.h: rows of the residual stream between two sub-layers."""
+    _fields_ = [("ids", c_void_p), ("table", c_void_p), ("ldt", c_longlong), ("vocab", c_int), ("table_f32", c_int), ("scale", c_float),
+                ("x", c_void_p), ("ldx", c_longlong), ("index", c_void_p), ("y", c_void_p), ("ldy", c_longlong), ("slot", c_void_p),
+                ("chosen", c_void_p), ("weight", c_void_p), ("top", c_int), ("experts", c_int), ("through", c_void_p),
+                ("ldt2", c_longlong), ("add", c_void_p), ("x_out", c_void_p), ("gain", c_float), ("eps", c_float), ("h", c_void_p),
+                ("ldh", c_longlong), ("f32", c_int), ("shift", c_void_p), ("state", c_void_p), ("state_ld", c_longlong),
+                ("num_seqs", c_int), ("positions", c_void_p), ("seq_ids", c_void_p), ("active", c_void_p), ("cu", c_void_p),
+                ("portions", c_int), ("max_len", c_int)]
+
+
+class LatentDims(ctypes.Structure):
+    """``b200_latent_dims`` of csrc/kernels/api.h."""
+    _fields_ = [("heads", c_int), ("rank", c_int), ("rot", c_int), ("true_rank", c_int), ("true_rot", c_int)]
 
 
 class PagedCacheDesc(ctypes.Structure):

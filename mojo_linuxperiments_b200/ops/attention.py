@@ -41,7 +41,7 @@ def rope_tables(max_pos: int, theta: float, device, head_dim: int = HEAD_DIM, ya
 
 class PagedKVCache:
     """One layer's paged KV storage, one record per page: [kv_heads][page_size][dk] keys, then
-    [kv_heads][page_size][dv] values (bf16, or fp32 for the 32-bit form of a model)."""
+    [kv_heads][page_size][dv] values (bf16, or fp32 for the 32-bit form of a model); dv = 0 for latents."""
 
     def __init__(self, num_pages: int, kv_heads: int, page_size: int, device, storage: torch.Tensor | None = None,
                  dk: int = HEAD_DIM, dv: int = HEAD_DIM, dtype: torch.dtype = torch.bfloat16):

@@ -57,7 +57,29 @@ class DynamicTanh:
         return DynamicTanh(float(alpha), vec(w), vec(b))
 
 
+@dataclass
+class GroupedW:
+    """Weights of several linears stacked row by row, [groups * n, k] with a padded row pitch."""
+    data: torch.Tensor
+    groups: int
+    n: int
+    k: int
+
+    @staticmethod
+    def of(ws, groups: int, dtype: torch.dtype, device, n: int | None = None) -> "GroupedW":
+        """``ws``: ``groups`` matrices [rows <= n, k], taken one at a time; missing rows are zero."""
+        data = None
+        for g, w in enumerate(ws):
+            rows_, k = w.shape
+            n = n or rows_
+            if data is None:
+                data = torch.zeros((groups * n, padded(k)), dtype=dtype, device=device)
+            data[g * n:g * n + rows_, :k] = w.to(device=device, dtype=dtype)
+        return GroupedW(data, groups, n, k)
+
+
 EPI_STORE, EPI_RESIDUAL, EPI_GLU = 0, 1, 2
+ACTIVATIONS = {None: 0, "relu2": 1}
 
 
 def _run(x: torch.Tensor, w: DenseW, epi, force: int = 0) -> None:
@@ -106,6 +128,54 @@ def linear_residual(x: torch.Tensor, w: DenseW, stream: torch.Tensor, mult: floa
                              norm_w=_lib.ptr(norm.w) if norm else None, norm_b=_lib.ptr(norm.b) if norm else None,
                              norm_alpha=norm.alpha if norm else 0.0)
     _run(x, w, epi, force)
+
+
+def linear_heads(x: torch.Tensor, w: GroupedW, x_group: int, y_group: int, gate: torch.Tensor | None = None,
+                 out_dtype: torch.dtype | None = None, splits: int = 0) -> torch.Tensor:
+    """One linear per head in one launch: group g takes columns g * x_group .. of x and writes columns g * y_group .. of the
+    result; ``gate`` fp32 [M, groups] (row stride free): logits of a sigmoid on each head's result."""
+    M = x.shape[0]
+    y = rows(M, w.groups * y_group, out_dtype or x.dtype, x.device)
+    if M == 0:
+        return y
+    assert x.dtype == w.data.dtype and x.stride(1) == 1 and x_group % 8 == 0 and y_group % 8 == 0 and y_group >= (w.n + 3) // 4 * 4
+    assert x.shape[1] >= (w.groups - 1) * x_group + w.k and (gate is None or gate.dtype == torch.float32)
+    epi = _lib.DenseEpilogue(mode=EPI_STORE, out_f32=int(y.dtype == torch.float32), exact=int(x.dtype == torch.float32), y=y.data_ptr(),
+                             ldy=y.stride(0), gate=_lib.ptr(gate), ldg=gate.stride(0) if gate is not None else 0, y_group=y_group)
+    g = _lib.GemmGroups(groups=w.groups, x_group=x_group)
+    if x.dtype == torch.float32:
+        rc = _lib.lib().b200_f32_gemm_grouped(x.data_ptr(), x.stride(0), w.data.data_ptr(), w.data.stride(0), M, w.n, w.k,
+                                              ctypes.byref(epi), ctypes.byref(g), _lib.stream())
+        _lib.check(rc, "f32_gemm_grouped")
+    else:
+        rc = _lib.lib().b200_bf16_gemm_decode_grouped(
+            x.data_ptr(), x.stride(0), w.data.data_ptr(), w.data.stride(0), M, M, w.n, w.k, ctypes.byref(epi), ctypes.byref(g),
+            default_workspace(x.device).status.data_ptr(), _lib.num_sms(x.device.index), splits, _lib.stream())
+        _lib.check(rc, "bf16_gemm_decode_grouped")
+    return y
+
+
+def linear_experts(x: torch.Tensor, w: GroupedW, work, act: str | None = None, force: int = 0) -> torch.Tensor:
+    """x: rows in the slot order of ``work`` (ops.moe.MoEWorkList); every expert multiplies its own rows."""
+    y = rows(x.shape[0], w.n, x.dtype, x.device)
+    if work.M == 0:
+        return y
+    assert x.dtype == w.data.dtype and x.stride(1) == 1 and x.shape[1] >= w.k and w.groups == work.n_local
+    f32 = int(x.dtype == torch.float32)
+    epi = _lib.DenseEpilogue(mode=EPI_STORE, out_f32=f32, exact=f32, y=y.data_ptr(), ldy=y.stride(0), act=ACTIVATIONS[act])
+    g = _lib.GemmGroups(groups=w.groups, offsets=work.offsets.data_ptr(), counts=work.counts.data_ptr(), tiles=work.tiles.data_ptr(),
+                        num_tiles=work.meta[1:].data_ptr(), max_tiles=work.max_tiles, expected=min(w.groups, work.max_slots))
+    args = (x.data_ptr(), x.stride(0), w.data.data_ptr(), w.data.stride(0))
+    if f32:
+        rc = _lib.lib().b200_f32_gemm_grouped(*args, work.M, w.n, w.k, ctypes.byref(epi), ctypes.byref(g), _lib.stream())
+        _lib.check(rc, "f32_gemm_grouped")
+        return y
+    tail = (ctypes.byref(epi), ctypes.byref(g), default_workspace(x.device).status.data_ptr(), _lib.num_sms(x.device.index), force, _lib.stream())
+    if work.M <= DECODE_MAX_M:
+        _lib.check(_lib.lib().b200_bf16_gemm_decode_grouped(*args, work.M, x.shape[0], w.n, w.k, *tail), "bf16_gemm_decode_grouped")
+    else:
+        _lib.check(_lib.lib().b200_bf16_gemm_grouped(*args, x.shape[0], w.n, w.k, *tail), "bf16_gemm_grouped")
+    return y
 
 
 def embed_norm(ids: torch.Tensor, table: torch.Tensor, d: int, scale: float, stream: torch.Tensor, copy: torch.Tensor | None,

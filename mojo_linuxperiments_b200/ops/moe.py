@@ -19,6 +19,18 @@ def router_topk(logits: torch.Tensor, k: int, renorm: bool = True):
     return ids, wts
 
 
+def route_grouped(logits: torch.Tensor, correction: torch.Tensor, top: int, groups: int, keep: int, scale: float, outputs: int):
+    """fp32 logits [M, >= outputs] -> (ids int32 [M, top], weights fp32 [M, top]).  softmax + ``correction`` decides who is
+    chosen, among the members of the best ``keep`` of ``groups`` equal groups; the weights are the softmax times ``scale``."""
+    M = logits.shape[0]
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1 and correction.dtype == torch.float32 and correction.numel() >= outputs
+    ids = torch.empty((M, top), dtype=torch.int32, device=logits.device)
+    wts = torch.empty((M, top), dtype=torch.float32, device=logits.device)
+    _lib.check(_lib.lib().b200_route_grouped(logits.data_ptr(), logits.stride(0), correction.data_ptr(), M, outputs, top, groups, keep,
+                                             float(scale), ids.data_ptr(), wts.data_ptr(), _lib.stream()), "route_grouped")
+    return ids, wts
+
+
 class MoEWorkList:
     """Device-side description of which (token, k) pairs this rank's experts process, in slot order."""
 
@@ -51,6 +63,15 @@ def moe_gather(xq: torch.Tensor, sx: torch.Tensor, w: MoEWorkList):
     _lib.check(_lib.lib().b200_moe_gather(xq.data_ptr(), sx.data_ptr(), d, w.slot_token.data_ptr(), w.meta.data_ptr(),
                                           w.max_slots, xp.data_ptr(), sp.data_ptr(), _lib.stream()), "moe_gather")
     return xp, sp
+
+
+def gather_rows(x: torch.Tensor, w: MoEWorkList) -> torch.Tensor:
+    """Rows of x (any element type, 16-byte row pitch) in slot order."""
+    out = torch.empty((w.max_slots, x.shape[1]), dtype=x.dtype, device=x.device)
+    assert x.is_contiguous()
+    _lib.check(_lib.lib().b200_moe_gather_rows(x.data_ptr(), x.stride(0) * x.element_size(), w.slot_token.data_ptr(), w.meta.data_ptr(),
+                                               w.max_slots, out.data_ptr(), _lib.stream()), "moe_gather_rows")
+    return out
 
 
 def grouped_gemm(xp: torch.Tensor, sp: torch.Tensor, wq: torch.Tensor, sw: torch.Tensor, w: MoEWorkList) -> torch.Tensor:

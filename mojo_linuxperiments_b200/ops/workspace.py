@@ -56,7 +56,8 @@ class Workspace:
             self.status.zero_()
             kernel = {0: "?", 1: "w8a8_gemm", 2: "w8a8_gemm_decode", 3: "attn_prefill", 4: "attn_decode_tma", 5: "attn_decode_tc",
                       6: "attn_decode_tcp", 7: "rope_kv_write", 8: "attn_decode", 9: "bf16_gemm", 10: "bf16_gemm_decode", 11: "attn_prefill_paged",
-                      12: "rotary_paged", 13: "attn_decode_paged", 14: "attn_paged"}.get(code >> 8, "?")
+                      12: "rotary_paged", 13: "attn_decode_paged", 14: "attn_paged",
+                      15: "latent_append", 16: "rotary_heads", 17: "latent_gather", 18: "attn_latent", 19: "attn_prefill_latent"}.get(code >> 8, "?")
             raise RuntimeError(f"kernel status {code & 255} in {kernel}: {_STATUS_NAMES.get(code & 255, 'unknown')}")
 
 
