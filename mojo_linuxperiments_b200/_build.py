@@ -37,7 +37,8 @@ KERNEL_LIB = "libb200_kernels.so"
 # "dense": production flags, but only the kernels of the unquantised (bf16 / fp32) models: what a tool that serves one
 # such model from a fresh checkout compiles.
 KERNEL_VARIANTS = {"": [], "trace": ["-DB200RT_TRACE"], "debug": ["-DB200RT_DEBUG"], "dense": []}
-KERNEL_SUBSETS = {"dense": ("attn_decode_paged.cu", "attn_paged.cu", "attn_prefill_paged.cu", "bf16_gemm.cu", "bf16_gemm_decode.cu",
+KERNEL_SUBSETS = {"dense": ("attn_decode_paged.cu", "attn_latent.cu", "attn_paged.cu", "attn_prefill_latent.cu",
+                            "attn_prefill_paged.cu", "bf16_gemm.cu", "bf16_gemm_decode.cu",
                             "f32_gemm.cu", "latent.cu", "mingru.cu", "moe.cu", "moe_route.cu", "rope_kv.cu", "rotary_paged.cu",
                             "stream_rows.cu", "tmap.cu", "trace.cu")}
 

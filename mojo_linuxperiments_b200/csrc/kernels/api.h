@@ -354,6 +354,21 @@ int b200_latent_gather(const b200_paged_cache* cache, const int* ctx, const int*
 int b200_attn_latent_any(const void* q, long long ldq, const void* q_rot, long long ldr, int head_ld_rot, void* out, long long ldo,
                          int M, const b200_latent_dims* dims, float scale, const int* positions, const int* seq_ids,
                          const int* seq_lens, const b200_paged_cache* cache, int* status, cudaStream_t stream);
+// bf16, page size 16, rank up to 512: q [M][heads][rank] (moved into the latent space), q_rot: first element of head 0's second
+// part, not yet turned, heads head_ld_rot apart.  Rows cu[b] .. cu[b+1] are consecutive positions of one sequence; cu NULL: one
+// token per sequence, seq_lens[b] = 0 marks an empty slot (zero output).  splits: CTAs (a cluster) that share the keys of a row tile.
+int b200_attn_latent_ctas_per_sm(int rank, int rot, int rows);
+int b200_attn_latent(const void* q, long long ldq, const void* q_rot, long long ldr, int head_ld_rot, void* out, long long ldo,
+                     int M, const b200_latent_dims* dims, float scale, const int* cu, int portions, int max_len, const int* positions,
+                     const int* seq_ids, const int* seq_lens, const float* cos_tab, const float* sin_tab, int max_pos,
+                     const b200_paged_cache* cache, int splits, int* status, cudaStream_t stream);
+// Long portions: q [M][heads][dn + dr] (turned) against expanded rows kv [rows][heads][dn] ++ [heads][dv] and the shared key part
+// k_rot [rows][dr]; rows ctx[b] .. ctx[b+1] are positions 0 .. of portion b's sequence.  gate: fp32 logits [M][heads] or NULL.
+int b200_attn_prefill_latent_fits(int dn, int dr, int dv);
+int b200_attn_prefill_latent(const void* q, long long ldq, int heads, int dn, int dr, int dv, const void* kv, long long ldkv,
+                             const void* k_rot, long long ldkr, int rows_kv, void* out, long long ldo, int M, int B, int max_len,
+                             float scale, const int* cu, const int* ctx, const int* positions, const float* gate, long long ldg,
+                             int* status, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

@@ -57,7 +57,7 @@ class LayeredDecoder:
         if isinstance(m, AttentionSpec):
             return X.Attention(m, self.dtype, self._tables)
         if isinstance(m, LatentSpec):
-            return X.LatentAttention(m, self.dtype, self._tables, self.cfg.eps)
+            return X.LatentAttention(m, self.dtype, self._tables, self.cfg.eps, self.rt.page_size)
         return X.MinGRU(m, self.dtype)
 
     def observe(self, run: int, x: torch.Tensor) -> None:

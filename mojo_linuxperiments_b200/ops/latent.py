@@ -6,7 +6,7 @@ import ctypes
 import torch
 
 from . import _lib
-from .attention import PagedKVCache
+from .attention import PAGE, PagedKVCache
 from .dense import rows
 from .workspace import default_workspace
 
@@ -62,4 +62,57 @@ def attend_any(q: torch.Tensor, q_rot: torch.Tensor, rot_head_ld: int, dm, scale
         q.data_ptr(), q.stride(0), q_rot.data_ptr(), q_rot.stride(0), rot_head_ld, out.data_ptr(), out.stride(0), q.shape[0],
         ctypes.byref(dm), float(scale), positions.data_ptr(), _lib.ptr(seq_ids), _lib.ptr(seq_lens), ctypes.byref(cache.desc(page_table)),
         _status(q), _lib.stream()), "attn_latent_any")
+    return out
+
+
+def fits(dm, dtype: torch.dtype, page_size: int, rows_per_portion: int = 32) -> bool:
+    """Whether ``attend`` takes these sizes (``attend_any`` takes all)."""
+    return (dtype == torch.bfloat16 and page_size == PAGE and
+            _lib.lib().b200_attn_latent_ctas_per_sm(dm.rank, dm.rot, rows_per_portion) > 0)
+
+
+def pick_splits(batch: int, row_tiles: int, keys: int, slots: int) -> int:
+    """CTAs per row tile: as many as still make one wave, with at least two tiles of 64 keys each."""
+    pairs, s = max(1, batch * row_tiles), 1
+    while s < 8 and pairs * s * 2 <= slots and keys // (2 * s) >= 128:
+        s *= 2
+    return s
+
+
+def attend(q: torch.Tensor, q_raw: torch.Tensor, raw_head_ld: int, dm, scale: float, positions: torch.Tensor, seq_ids: torch.Tensor | None,
+           cos: torch.Tensor, sin: torch.Tensor, cache: PagedKVCache, page_table: torch.Tensor, *, cu: torch.Tensor | None = None,
+           max_len: int = 1, seq_lens: torch.Tensor | None = None, keys: int | None = None, splits: int | None = None) -> torch.Tensor:
+    """bf16: q [M, heads * rank] against the latents, q_raw (its second part, not yet turned) against the key parts -> weighted
+    latents [M, heads * rank].  ``cu``: portions of consecutive tokens; None: one token per sequence.  ``keys``: most keys a
+    row sees (default: what the page table can hold)."""
+    M = q.shape[0]
+    out = rows(M, dm.heads * dm.rank, q.dtype, q.device)
+    if splits is None:
+        longest, batch = (int(max_len), cu.numel() - 1) if cu is not None else (1, M)
+        per_cta = 32 if longest * dm.heads > 16 else 16
+        slots = _lib.num_sms(q.device.index) * _lib.lib().b200_attn_latent_ctas_per_sm(dm.rank, dm.rot, per_cta)
+        splits = pick_splits(batch, -(-longest * dm.heads // per_cta), keys or page_table.shape[1] * cache.page_size, slots)
+    _lib.check(_lib.lib().b200_attn_latent(
+        q.data_ptr(), q.stride(0), q_raw.data_ptr(), q_raw.stride(0), raw_head_ld, out.data_ptr(), out.stride(0), M, ctypes.byref(dm),
+        float(scale), _lib.ptr(cu), cu.numel() - 1 if cu is not None else 0, int(max_len), positions.data_ptr(), _lib.ptr(seq_ids),
+        _lib.ptr(seq_lens), cos.data_ptr(), sin.data_ptr(), cos.shape[0], ctypes.byref(cache.desc(page_table)), splits, _status(q),
+        _lib.stream()), "attn_latent")
+    return out
+
+
+def expanded_fits(dn: int, dr: int, dv: int) -> bool:
+    return bool(_lib.lib().b200_attn_prefill_latent_fits(dn, dr, dv))
+
+
+def attend_expanded(q: torch.Tensor, heads: int, dn: int, dr: int, dv: int, kv: torch.Tensor, k_rot: torch.Tensor, scale: float,
+                    cu: torch.Tensor, ctx: torch.Tensor, positions: torch.Tensor, max_len: int, gate: torch.Tensor | None = None) -> torch.Tensor:
+    """q [M, heads * (dn + dr)] (turned) against kv [rows, heads * dn + heads * dv] and k_rot [rows, >= dr], rows ctx[b] .. of
+    portion b's sequence from its first token on -> [M, heads * dv], times the sigmoid of ``gate`` fp32 [M, heads]."""
+    M = q.shape[0]
+    out = rows(M, heads * dv, q.dtype, q.device)
+    assert gate is None or gate.dtype == torch.float32
+    _lib.check(_lib.lib().b200_attn_prefill_latent(
+        q.data_ptr(), q.stride(0), heads, dn, dr, dv, kv.data_ptr(), kv.stride(0), k_rot.data_ptr(), k_rot.stride(0), kv.shape[0],
+        out.data_ptr(), out.stride(0), M, cu.numel() - 1, int(max_len), float(scale), cu.data_ptr(), ctx.data_ptr(), positions.data_ptr(),
+        _lib.ptr(gate), gate.stride(0) if gate is not None else 0, _status(q), _lib.stream()), "attn_prefill_latent")
     return out
