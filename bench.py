@@ -2,7 +2,7 @@
 
     python bench.py --gpus N --steps K --warmup W            (N > 1: launched by torch.distributed.run, one rank per GPU)
     python bench.py --impl reference ...                     (prints why the Mojo reference cannot run here)
-    python bench.py --layered                                (Volonex beside the W8A8 decoder of equal size, kernel by kernel)
+    python bench.py --layered [volonex|rakelorn]             (a layer-by-layer design beside its closest model, kernel by kernel)
     python bench.py --impl torch_baseline ...                (PyTorch + cuBLAS int8 + NCCL build of the same model)
 
 One step = one decode step of the whole batch (32 sequences, 1,024-token prompts already in the paged KV cache), so
@@ -45,7 +45,8 @@ def parse():
     ap.add_argument("--skip-self-check", action="store_true", help="do not decode the miniature model against the oracle before timing")
     ap.add_argument("--metrics-log", default=os.path.join(tempfile.gettempdir(), "b200rt_bench_metrics.jsonl"),
                     help="append the result record to this JSON-lines file (empty: do not)")
-    ap.add_argument("--layered", action="store_true", help="instead of the headline workload: the Volonex design beside the W8A8 decoder of equal size (one GPU)")
+    ap.add_argument("--layered", nargs="?", const="volonex", choices=["volonex", "rakelorn"], help="instead of the headline workload: a "
+                    "layer-by-layer design beside the closest models of equal size (one GPU)")
     ap.add_argument("--layers", type=int, default=0, help="smoke runs only: override the layer count (the line is then marked invalid)")
     return ap.parse_args()
 
@@ -482,11 +483,11 @@ def main():
                           "'not installable'; no mojo/pixi toolchain offline) and has no model, decode or GPU path to run this metric"}))
         return
     if args.layered:
-        from benchmarks import bench_layered
+        from benchmarks import bench_layered, bench_rakelorn
         torch.cuda.set_device(0)
         sampler = ClockSampler(0)
         sampler.mark_start()
-        result = bench_layered.run()
+        result = (bench_rakelorn if args.layered == "rakelorn" else bench_layered).run()
         result["clocks"] = sampler.stop()
         print(json.dumps(result), flush=True)
         return
