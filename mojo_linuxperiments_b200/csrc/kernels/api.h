@@ -357,7 +357,7 @@ int b200_attn_latent_any(const void* q, long long ldq, const void* q_rot, long l
 // bf16, page size 16, rank up to 512: q [M][heads][rank] (moved into the latent space), q_rot: first element of head 0's second
 // part, not yet turned, heads head_ld_rot apart.  Rows cu[b] .. cu[b+1] are consecutive positions of one sequence; cu NULL: one
 // token per sequence, seq_lens[b] = 0 marks an empty slot (zero output).  splits: CTAs (a cluster) that share the keys of a row tile.
-int b200_attn_latent_ctas_per_sm(int rank, int rot, int rows);
+int b200_attn_latent_fits(int rank, int rot);
 int b200_attn_latent(const void* q, long long ldq, const void* q_rot, long long ldr, int head_ld_rot, void* out, long long ldo,
                      int M, const b200_latent_dims* dims, float scale, const int* cu, int portions, int max_len, const int* positions,
                      const int* seq_ids, const int* seq_lens, const float* cos_tab, const float* sin_tab, int max_pos,

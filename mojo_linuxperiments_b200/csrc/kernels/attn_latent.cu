@@ -1,82 +1,100 @@
-// Latent attention over the paged cache in the latent space (bf16): queries that were moved there against the cached latents
-// and the shared rotated key part, for decoding and for short portions.  All heads read the same keys, and a key's first
-// `rank` dimensions are also its value, so a cached row is fetched once for scores and values.
+// Latent attention over the paged cache in the latent space (bf16, tcgen05): queries that were moved there against the cached
+// latents and the shared rotated key part, for decoding and for short portions.  All heads read the same keys and a key's first
+// `rank` dimensions are also its value, so a cached row is fetched once, by TMA, and serves both products from shared memory.
 //
-// Rows are (token, head) pairs of one portion in order; a CTA takes 16 or 32 of them against 64 keys at a time.  The op is
-// bound by the cached bytes for a few heads, so a tile of 64 rows (up to 80 KB) is in flight while the one before is
-// computed.  The eight warps share a tile: scores by keys (8 each, m16n8k16 MMAs over the whole row), softmax by rows through
-// shared memory, values by columns (16-column units), so no warp holds more than its part of the accumulators.  The splits of
-// one row tile are a thread-block cluster that merges through distributed shared memory.  The rotary embedding of the query's
-// second part happens while it is loaded.
+// Rows are (token, head) pairs of one portion in order, N = 16 or 32 of them per CTA.  So few rows would waste the MMA's 128, so
+// the keys take that side:  S^T [128 keys, N] = C [128, dk] . Q^T,   O^T [rank, N] = C^T [rank, 128] . P^T in blocks of 128 value
+// dimensions - the same operand tile, once K-major and once MN-major.
+//   warp 0      TMA producer: a tile is 128 keys = 8 pages, in slots of 128 latent columns and one of the rotated part, each
+//               released as soon as its last product is done (rings; a tile of 512 + 64 columns is 144 KB, so the next one
+//               streams in as this one leaves).  In decoding the tiles of earlier tokens are requested before the dependency
+//               wait: only the new token's row is written by a kernel that may still run.
+//   warp 1      MMA issuer; where two tiles fit, the scores of the next tile go before the values of this one
+//   warps 2..9  softmax with keys on the lanes: a warp holds 32 keys of half the rows; maxima by warp reduction and through
+//               shared memory, sums stay with their keys until the end.  They also turn the queries' second part, and keep the
+//               accumulated values (128 dimensions x N per block) in registers.
+// The splits of one row tile are a thread-block cluster that merges through distributed shared memory.  All waits are bounded.
 #include "ptx.cuh"
 #include "api.h"
 #include "launch.cuh"
+#include "gemm_common.cuh"
 
 namespace b200 {
 
-constexpr int AL_THREADS = 256, AL_KEYS = 64, AL_PS = 16, AL_PP = AL_KEYS + 8, AL_SP = AL_KEYS + 4;
+constexpr int AL_THREADS = 320, AL_SOFTMAX = 256, AL_KEYS = 128, AL_PS = 16;
+constexpr int AL_CHUNK = 128 * 128;                  // 128 keys x 64 bf16
+constexpr int AL_SLOT = 2 * AL_CHUNK;                // 128 latent columns
+constexpr int AL_MAX_SMEM = 232448, AL_MAX_SLOTS = 8;
 constexpr float AL_LOG2E = 1.4426950408889634f;
-constexpr int AL_MAX_SMEM = 232448;
 
 struct AttnLatentParams {
-  const __nv_bfloat16* q; long long ldq;
   const __nv_bfloat16* q_rot; long long ldr; int head_ld_rot;
   __nv_bfloat16* out; long long ldo;
   b200_latent_dims d;
   float scale_log2;
   const int* cu; const int* positions; const int* seq_ids; const int* seq_lens;
   const float* cos_tab; const float* sin_tab;
-  int max_pos, splits;
+  int max_pos, splits, slots, rot_slots, ahead;
   b200_paged_cache c;
   int* status;
+  unsigned long long limit_ns;
 };
 
-__device__ __forceinline__ void al_cp16(uint32_t dst, const void* src, bool valid) {
-  const int n = valid ? 16 : 0;      // 0 source bytes: the destination is filled with zeros
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
-__device__ __forceinline__ void al_ldm(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void al_ldm_t(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void al_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 __device__ __forceinline__ float al_ld_cluster(uint32_t addr) {
   float v;
   asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
   return v;
 }
-
-// shared memory: two tiles of keys, the queries, softmax weights, scores, per-row numbers; the key tiles become the merge buffer
-__host__ __device__ inline int al_kp(int dk) { return ((dk + 15) / 16) * 16 + 8; }      // row pitch: 16-byte skew, ldmatrix without conflicts
-__host__ __device__ inline int al_smem(int dk, int mt) {
-  const int kp = al_kp(dk);
-  return 2 * AL_KEYS * kp * 2 + 16 * mt * (kp * 2 + AL_PP * 2 + AL_SP * 4) + 16 * mt * 4 * (3 + 8);
+__device__ __forceinline__ float4 al_ld_cluster4(uint32_t addr) {
+  float4 v;
+  asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
+  return v;
+}
+// integers in the order of the floats they come from
+__device__ __forceinline__ int al_order(int i) { return i ^ ((i >> 31) & 0x7fffffff); }
+__device__ __forceinline__ float al_warp_max(float v) {
+  return __int_as_float(al_order(__reduce_max_sync(0xffffffffu, al_order(__float_as_int(v)))));
+}
+// element (row, key) of a K-major operand with 128-byte swizzle: rows of 64 elements, eight rows per 1024 bytes
+__device__ __forceinline__ uint32_t al_swizzled(int row, int col) {
+  return (row >> 3) * 1024 + (row & 7) * 128 + (((col >> 3) ^ (row & 7)) << 4) + (col & 7) * 2;
 }
 
-template <int MT, int NU>
-__global__ void __launch_bounds__(AL_THREADS, NU == 4 ? 1 : 2)
-attn_latent_kernel(const __grid_constant__ AttnLatentParams p) {
-  constexpr int ROWS = 16 * MT, TPR = AL_THREADS / ROWS, KPT = AL_KEYS / TPR;      // softmax: threads per row, keys per thread
+template <int N>
+struct AlShared {      // behind the operands
+  float red[2][4][N];  // maxima of the four key quarters, two turns
+  float alpha[2][N];
+  float m[N], l[N], lw[4][N];
+  float f[8][N];       // factor of every split
+  int pos[N];
+  uint64_t bars[2 * AL_MAX_SLOTS + 16];
+  uint32_t tmem;
+  int abort;
+};
+
+template <int N>
+__global__ void __launch_bounds__(AL_THREADS, 1)
+attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_c,
+                   const __grid_constant__ CUtensorMap tmap_r, const __grid_constant__ AttnLatentParams p) {
+  constexpr int NC = N / 2;                              // columns of a softmax thread
+  constexpr int QCHUNK = N * 128, TMEM_COLS = N == 32 ? 512 : 256, TMEM_O = 2 * N;
   pdl_launch_dependents();
-  pdl_wait();
-  extern __shared__ __align__(128) uint8_t al_smem_raw[];
+  if (p.cu) pdl_wait();                                  // decoding: page table, positions and earlier rows are older than this step
+  extern __shared__ __align__(1024) uint8_t al_smem[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int H = p.d.heads, rank = p.d.rank, rot = p.d.rot, dk = rank + rot, ks = (dk + 15) >> 4, KP = al_kp(dk);
-  const int b = blockIdx.z, S = p.splits, split = blockIdx.x, g0 = blockIdx.y * ROWS;
+  const int H = p.d.heads, rank = p.d.rank, rot = p.d.rot;
+  const int nd = (rank + 127) >> 7, kq = (rank + 63) >> 6, rc = (rot + 63) >> 6;      // slots per tile, chunks of each part
+  const int b = blockIdx.z, S = p.splits, split = blockIdx.x, g0 = blockIdx.y * N;
   const int row0 = p.cu ? p.cu[b] : b, len = p.cu ? p.cu[b + 1] - row0 : 1;
   if (g0 >= len * H) return;                             // the same for all CTAs of the cluster, as below
-  const int n_rows = min(ROWS, len * H - g0);
+  const int n_rows = min(N, len * H - g0);
   const int start = p.positions[row0], seq = p.seq_ids ? p.seq_ids[row0] : b;
   const int last_pos = start + (g0 + n_rows - 1) / H;
   const bool empty = p.seq_lens && p.seq_lens[b] <= 0;
   const bool bad = start < 0 || last_pos >= p.max_pos || seq < 0 || seq >= p.c.num_seqs || last_pos / AL_PS >= p.c.max_pages;
   if (empty || bad) {
     if (bad && tid == 0 && p.status) atomicCAS(p.status, 0, static_cast<int>(ST_BAD_ARGUMENT) | (18 << 8));
+    pdl_wait();
     if (split == 0)
       for (int i = tid; i < n_rows * rank; i += AL_THREADS) {
         const int g = g0 + i / rank, tok = g / H;
@@ -84,226 +102,339 @@ attn_latent_kernel(const __grid_constant__ AttnLatentParams p) {
       }
     return;
   }
-  const int stage_bytes = AL_KEYS * KP * 2;
-  uint8_t* s_q = al_smem_raw + 2 * stage_bytes;
-  __nv_bfloat16* s_p = reinterpret_cast<__nv_bfloat16*>(s_q + ROWS * KP * 2);
-  float* s_s = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(s_p) + ROWS * AL_PP * 2);
-  float* s_alpha = s_s + ROWS * AL_SP;                   // [ROWS], then the row's maximum and sum, then a factor per split
-  float* s_m = s_alpha + ROWS;
-  float* s_l = s_m + ROWS;
-  float* s_f = s_l + ROWS;
-  const uint32_t ring = smem_u32(al_smem_raw);
+  const uint32_t sC = smem_u32(al_smem), sR = sC + p.slots * AL_SLOT, sQ = sR + p.rot_slots * rc * AL_CHUNK, sP = sQ + (kq + rc) * QCHUNK;
+  uint8_t* pQr = al_smem + (sQ - sC) + kq * QCHUNK;
+  uint8_t* pP = al_smem + (sP - sC);
+  AlShared<N>& sh = *reinterpret_cast<AlShared<N>*>(pP + (p.ahead ? 2 : 1) * 2 * QCHUNK);
+  const uint32_t bar0 = smem_u32(sh.bars);
+  enum { B_Q = 0, B_QROT = 1, B_SFULL = 2, B_PFULL = 4, B_OFULL = 5, B_RFULL = 7, B_REMPTY = 9, B_CFULL = 11, B_CEMPTY = 11 + AL_MAX_SLOTS, B_COUNT = 11 + 2 * AL_MAX_SLOTS };
+  auto bar = [&](int i) { return bar0 + 8u * i; };
+  volatile int* abort_flag = &sh.abort;
+  const uint64_t limit = p.limit_ns;
 
   const int n_tiles = last_pos / AL_KEYS + 1;
-  const int ta = static_cast<int>(static_cast<long long>(n_tiles) * split / S), tb = static_cast<int>(static_cast<long long>(n_tiles) * (split + 1) / S);
-  const int* pt = p.c.page_table + static_cast<size_t>(seq) * p.c.max_pages;
-  const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(p.c.data);
-  const int kc = dk >> 3, r_first = lane / kc, c_first = lane - r_first * kc, r_step = 32 / kc, c_step = 32 - r_step * kc;
-  // a warp fetches eight consecutive rows, half a page: one contiguous run
-  auto issue = [&](int t, int st) {
-    const int key0 = t * AL_KEYS + warp * 8, left = last_pos + 1 - key0;
-    const int page = left > 0 ? pt[key0 / AL_PS] : -1;
-    const bool ok = page >= 0 && page < p.c.num_pages;
-    const __nv_bfloat16* src = cache + (ok ? (static_cast<size_t>(page) * AL_PS + key0 % AL_PS) * dk : 0) + lane * 8;
-    const uint32_t dst = ring + st * stage_bytes + warp * 8 * KP * 2;
-    for (int r = r_first, c = c_first; r < 8; src += 256) {
-      al_cp16(dst + (r * KP + c * 8) * 2, ok ? src : cache, ok && r < left);
-      r += r_step; c += c_step;
-      if (c >= kc) { c -= kc; ++r; }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  if (ta < tb) issue(ta, 0);
+  const int ta = static_cast<int>(static_cast<long long>(n_tiles) * split / S), nt = static_cast<int>(static_cast<long long>(n_tiles) * (split + 1) / S) - ta;
 
-  // columns dk .. of the key rows are never fetched: zero once
-  if (dk & 15)
-    for (int i = tid; i < 2 * AL_KEYS; i += AL_THREADS) *reinterpret_cast<uint4*>(al_smem_raw + (i * KP + dk) * 2) = make_uint4(0u, 0u, 0u, 0u);
-  for (int i = tid; i < ROWS * ks * 2; i += AL_THREADS) {
-    const int r = i / (ks * 2), c = (i - r * ks * 2) * 8, g = g0 + r, tok = g / H;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < n_rows && c < rank) v = *reinterpret_cast<const uint4*>(p.q + static_cast<size_t>(row0 + tok) * p.ldq + static_cast<size_t>(g - tok * H) * rank + c);
-    if (c < rank || c >= dk) *reinterpret_cast<uint4*>(s_q + (r * KP + c) * 2) = v;
+  if (tid == 0) {
+    for (int i = 0; i < B_COUNT; ++i) mbar_init(bar(i), i == B_PFULL || i == B_QROT ? AL_SOFTMAX : 1);
+    *abort_flag = 0;
+    mbar_fence_init();
   }
-  const int np = p.d.true_rot / 2;
-  for (int i = tid; i < ROWS * (rot / 2); i += AL_THREADS) {
-    const int r = i / (rot / 2), j = i - r * (rot / 2), g = g0 + r, tok = g / H;
-    float u = 0.f, v = 0.f;
-    if (r < n_rows && j < np) {
-      const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(p.q_rot + static_cast<size_t>(row0 + tok) * p.ldr + static_cast<size_t>(g - tok * H) * p.head_ld_rot + 2 * j);
-      const float c = p.cos_tab[static_cast<size_t>(start + tok) * np + j], s = p.sin_tab[static_cast<size_t>(start + tok) * np + j];
-      const float a = __low2float(x), d = __high2float(x);
-      u = a * c - d * s;
-      v = d * c + a * s;
+  if (tid < N) sh.pos[tid] = start + min(g0 + tid, len * H - 1) / H;
+  if (warp == 1) { tmem_alloc(smem_u32(&sh.tmem), TMEM_COLS); tmem_relinquish(); }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = sh.tmem;
+
+  float o[2][N];                                         // softmax warps: value dimensions x rows, blocks half and half + 2
+#pragma unroll
+  for (int i = 0; i < N; ++i) o[0][i] = o[1][i] = 0.f;
+
+  if (warp == 0) {
+    const int* pt = p.c.page_table + static_cast<size_t>(seq) * p.c.max_pages;
+    auto page_of = [&](int t) {                          // lane <-> page of tile t; past the last key: out of range, arrives as zeros
+      const int tok = t * AL_KEYS + (lane & 7) * AL_PS;
+      const int pg = tok <= last_pos ? pt[tok / AL_PS] : p.c.num_pages;
+      return pg < 0 || pg > p.c.num_pages ? p.c.num_pages : pg;
+    };
+    if (lane == 0) { prefetch_tmap(&tmap_c); prefetch_tmap(&tmap_r); }
+    bool waited = p.cu != nullptr, ok = true;
+    int cs = 0, rs = 0;
+    uint32_t cp = 0, rp = 0;
+    int page = nt > 0 ? page_of(ta) : 0;
+    for (int j = 0; j < nt && ok; ++j) {
+      if (!waited && (ta + j + 1) * AL_KEYS > last_pos) { pdl_wait(); waited = true; }      // holds the new token
+      const int next = j + 1 < nt ? page_of(ta + j + 1) : 0;
+      for (int d = 0; d < nd; ++d) {
+        const int chunks = min(2, kq - 2 * d);
+        ok = __all_sync(0xffffffffu, mbar_wait(bar(B_CEMPTY + cs), cp ^ 1u, abort_flag, p.status, (ST_TIMEOUT_SMEM_EMPTY | (18 << 8)), limit));
+        if (!ok) break;
+        if (lane == 0) mbar_expect_tx(bar(B_CFULL + cs), chunks * AL_CHUNK);
+        __syncwarp();
+        // lanes 0..7 fetch the first chunk's pages, 8..15 the second's
+        if (lane < 8 * chunks)
+          tma_load_3d(sC + cs * AL_SLOT + (lane >> 3) * AL_CHUNK + (lane & 7) * 2048, &tmap_c, bar(B_CFULL + cs), (2 * d + (lane >> 3)) * 64, 0, page);
+        if (++cs == p.slots) { cs = 0; cp ^= 1u; }
+      }
+      if (ok && rc > 0) {
+        ok = __all_sync(0xffffffffu, mbar_wait(bar(B_REMPTY + rs), rp ^ 1u, abort_flag, p.status, (ST_TIMEOUT_SMEM_EMPTY | (18 << 8)), limit));
+        if (!ok) break;
+        if (lane == 0) mbar_expect_tx(bar(B_RFULL + rs), rc * AL_CHUNK);
+        __syncwarp();
+        if (lane < 8 * rc)
+          tma_load_3d(sR + rs * rc * AL_CHUNK + (lane >> 3) * AL_CHUNK + (lane & 7) * 2048, &tmap_r, bar(B_RFULL + rs), (lane >> 3) * 64, 0, page);
+        if (++rs == p.rot_slots) { rs = 0; rp ^= 1u; }
+      }
+      page = next;
     }
-    *reinterpret_cast<__nv_bfloat162*>(s_q + (r * KP + rank + 2 * j) * 2) = __floats2bfloat162_rn(u, v);
-  }
-
-  float o[MT][2 * NU][4];
-#pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int i = 0; i < 2 * NU; ++i)
-#pragma unroll
-      for (int k = 0; k < 4; ++k) o[mt][i][k] = 0.f;
-  // this thread's share of the softmax
-  const int my_row = tid / TPR, my_key = (tid % TPR) * KPT;
-  const int my_pos = start + min(g0 + my_row, len * H - 1) / H;
-  float m_run = -INFINITY, l_run = 0.f;
-  const uint32_t a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;      // ldmatrix rows / columns of an A operand
-
-  for (int t = ta; t < tb; ++t) {
-    const uint32_t kt = ring + ((t - ta) & 1) * stage_bytes;
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                     // tile t is in for everyone; everyone is done with tile t - 1
-    if (t + 1 < tb) issue(t + 1, (t + 1 - ta) & 1);
-    float s[MT][2][4];
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int i = 0; i < 2; ++i)
-#pragma unroll
-        for (int k = 0; k < 4; ++k) s[mt][i][k] = 0.f;
-    const uint32_t ka = kt + ((warp * 8 + (lane & 7)) * KP + (lane >> 3) * 8) * 2;
-    const uint32_t qa0 = smem_u32(s_q) + (a_row * KP + a_col) * 2;
-#pragma unroll 4
-    for (int kk = 0; kk < ks; kk += 2) {
-      uint32_t kb[4];
-      al_ldm(ka + kk * 32, kb);                          // keys x 32 dimensions (the last 16 unused when ks is odd)
-#pragma unroll
-      for (int mt = 0; mt < MT; ++mt) {
-        uint32_t qa[4];
-        al_ldm(qa0 + mt * 16 * KP * 2 + kk * 32, qa);
-        al_mma(s[mt][0], qa, kb[0], kb[1]);
-        if (kk + 1 < ks) {
-          al_ldm(qa0 + mt * 16 * KP * 2 + kk * 32 + 32, qa);
-          al_mma(s[mt][1], qa, kb[2], kb[3]);
+    if (!ok) { const uint64_t t0 = globaltimer_ns(); while (globaltimer_ns() - t0 < 2000000ull) { } }   // copies in flight land
+    if (!waited) pdl_wait();
+    __syncwarp();
+  } else if (warp == 1) {
+    pdl_wait();
+    if (lane == 0 && nt > 0) {
+      constexpr uint32_t IDESC_S = umma_idesc_bf16(128, N, 0, 0), IDESC_O = umma_idesc_bf16(128, N, 1, 0);      // C^T is MN-major
+      mbar_expect_tx(bar(B_Q), kq * QCHUNK);
+      for (int c = 0; c < kq; ++c) tma_load_3d(sQ + c * QCHUNK, &tmap_q, bar(B_Q), c * 64, row0 * H + g0, 0);
+      const int c_steps = (rank + 15) >> 4, r_steps = (rot + 15) >> 4;
+      int cs = 0, rs = 0, vs = 0;                        // slots: scores read cs, values vs
+      uint32_t cp = 0, rp = 0;
+      auto issue_s = [&](int j) -> bool {
+        const uint32_t d_tmem = tmem_base + (j & 1) * N;
+        uint32_t acc = 0;
+        for (int d = 0; d < nd; ++d) {
+          if (!mbar_wait(bar(B_CFULL + cs), cp, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (18 << 8)), limit)) return false;
+          tc_fence_after();
+          const int steps = min(8, c_steps - 8 * d);
+          for (int kk = 0; kk < steps; ++kk, acc = 1)
+            umma_f16_ss(d_tmem, umma_desc_k_sw128(sC + cs * AL_SLOT + (kk >> 2) * AL_CHUNK) + 2ull * (kk & 3),
+                        umma_desc_k_sw128(sQ + (2 * d + (kk >> 2)) * QCHUNK) + 2ull * (kk & 3), IDESC_S, acc);
+          if (++cs == p.slots) { cs = 0; cp ^= 1u; }
         }
+        if (rc > 0) {
+          if (!mbar_wait(bar(B_RFULL + rs), rp, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (18 << 8)), limit)) return false;
+          tc_fence_after();
+          for (int kk = 0; kk < r_steps; ++kk, acc = 1)
+            umma_f16_ss(d_tmem, umma_desc_k_sw128(sR + (rs * rc + (kk >> 2)) * AL_CHUNK) + 2ull * (kk & 3),
+                        umma_desc_k_sw128(sQ + (kq + (kk >> 2)) * QCHUNK) + 2ull * (kk & 3), IDESC_S, acc);
+          umma_commit(bar(B_REMPTY + rs));
+          if (++rs == p.rot_slots) { rs = 0; rp ^= 1u; }
+        }
+        umma_commit(bar(B_SFULL + (j & 1)));
+        return true;
+      };
+      bool ok = mbar_wait(bar(B_Q), 0, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (18 << 8)), limit) &&
+                mbar_wait(bar(B_QROT), 0, abort_flag, p.status, (ST_TIMEOUT_PEER_FLAG | (18 << 8)), limit);
+      if (ok) { tc_fence_after(); ok = issue_s(0); }
+      for (int j = 0; j < nt && ok; ++j) {
+        if (p.ahead && j + 1 < nt && !issue_s(j + 1)) { ok = false; break; }
+        if (!mbar_wait(bar(B_PFULL), j & 1u, abort_flag, p.status, (ST_TIMEOUT_PEER_FLAG | (18 << 8)), limit)) { ok = false; break; }
+        tc_fence_after();
+        const uint32_t pd = sP + (p.ahead ? (j & 1) * 2 * QCHUNK : 0);
+        for (int d = 0; d < nd; ++d) {
+          const uint32_t d_tmem = tmem_base + TMEM_O + ((j & 1) * 4 + d) * N;
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk)
+            umma_f16_ss(d_tmem, umma_desc_mn_sw128(sC + vs * AL_SLOT + kk * 2048, AL_CHUNK, 1024),
+                        umma_desc_k_sw128(pd + (kk >> 2) * QCHUNK) + 2ull * (kk & 3), IDESC_O, kk > 0 ? 1u : 0u);
+          umma_commit(bar(B_CEMPTY + vs));
+          if (++vs == p.slots) vs = 0;
+        }
+        umma_commit(bar(B_OFULL + (j & 1)));
+        if (!p.ahead && j + 1 < nt && !issue_s(j + 1)) { ok = false; break; }
       }
     }
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
-      float* at = s_s + (mt * 16 + (lane >> 2)) * AL_SP + warp * 8 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(at) = make_float2(s[mt][0][0] + s[mt][1][0], s[mt][0][1] + s[mt][1][1]);
-      *reinterpret_cast<float2*>(at + 8 * AL_SP) = make_float2(s[mt][0][2] + s[mt][1][2], s[mt][0][3] + s[mt][1][3]);
+    __syncwarp();
+  } else {
+    pdl_wait();
+    const int qd = warp & 3, half = (warp - 2) >> 2, c0 = half * NC;      // key quarter = TMEM lane quarter; first column
+    const int st = tid - 64;
+    // the queries' rotated part; columns up to the end of its chunks and rows beyond the portion are zero
+    const int np = p.d.true_rot / 2, wide = rc * 32;
+    for (int i = st; i < N * wide; i += AL_SOFTMAX) {
+      const int r = i / wide, j = i - r * wide, g = g0 + r, tok = g / H;
+      float u = 0.f, v = 0.f;
+      if (r < n_rows && j < np) {
+        const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(p.q_rot + static_cast<size_t>(row0 + tok) * p.ldr + static_cast<size_t>(g - tok * H) * p.head_ld_rot + 2 * j);
+        const float c = p.cos_tab[static_cast<size_t>(start + tok) * np + j], s = p.sin_tab[static_cast<size_t>(start + tok) * np + j];
+        const float a = __low2float(x), e = __high2float(x);
+        u = a * c - e * s;
+        v = e * c + a * s;
+      }
+      *reinterpret_cast<__nv_bfloat162*>(pQr + (j >> 5) * QCHUNK + al_swizzled(r, (2 * j) & 63)) = __floats2bfloat162_rn(u, v);
     }
-    __syncthreads();
-    {
-      float v[KPT], mx = -INFINITY;
+    fence_proxy_async_smem();
+    mbar_arrive(bar(B_QROT));
+
+    const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(qd * 32) << 16);
+    float m_run[NC], l_run[NC];
 #pragma unroll
-      for (int i = 0; i < KPT; i += 4) {
-        const float4 x = *reinterpret_cast<const float4*>(s_s + my_row * AL_SP + my_key + i);
-        v[i] = x.x; v[i + 1] = x.y; v[i + 2] = x.z; v[i + 3] = x.w;
-      }
+    for (int i = 0; i < NC; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+    bool ok = true;
+    auto wait_all = [&](int i, uint32_t par) {           // one verdict per warp: the TMEM loads need all lanes
+      return __all_sync(0xffffffffu, mbar_wait(bar(i), par, abort_flag, p.status, (ST_TIMEOUT_TMEM_FULL | (18 << 8)), limit)) != 0;
+    };
+    auto o_update = [&](int j) -> bool {
+      if (!wait_all(B_OFULL + (j & 1), (j >> 1) & 1u)) return false;
+      tc_fence_after();
+      const float4* al = reinterpret_cast<const float4*>(sh.alpha[j & 1]);
 #pragma unroll
-      for (int i = 0; i < KPT; ++i) {
-        v[i] = t * AL_KEYS + my_key + i <= my_pos ? v[i] * p.scale_log2 : -INFINITY;
-        mx = fmaxf(mx, v[i]);
-      }
+      for (int k = 0; k < 2; ++k) {
+        const int d = half + 2 * k;
+        if (d < nd) {
+          uint32_t v[N];
+          if constexpr (N == 32) tmem_ld_x32(t_lane + TMEM_O + ((j & 1) * 4 + d) * N, v);
+          else tmem_ld_x16(t_lane + TMEM_O + ((j & 1) * 4 + d) * N, v);
+          tmem_ld_wait();
 #pragma unroll
-      for (int w = TPR / 2; w > 0; w >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
-      const float m_new = fmaxf(m_run, mx), m_use = m_new == -INFINITY ? 0.f : m_new;
-      const float alpha = m_run == -INFINITY ? 0.f : exp2f(m_run - m_use);
-      m_run = m_new;
-      float sum = 0.f;
-      uint32_t pk[KPT / 2];
-#pragma unroll
-      for (int i = 0; i < KPT; i += 2) {
-        const __nv_bfloat162 e = __floats2bfloat162_rn(exp2f(v[i] - m_use), exp2f(v[i + 1] - m_use));
-        sum += __low2float(e) + __high2float(e);         // what the MMA will actually see
-        pk[i / 2] = *reinterpret_cast<const uint32_t*>(&e);
-      }
-#pragma unroll
-      for (int i = 0; i < KPT / 2; i += 2) *reinterpret_cast<uint2*>(s_p + my_row * AL_PP + my_key + 2 * i) = make_uint2(pk[i], pk[i + 1]);
-      l_run = l_run * alpha + sum;
-      if (my_key == 0) s_alpha[my_row] = alpha;
-    }
-    __syncthreads();
-    uint32_t pa[MT][4][4];
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
-      const float f0 = s_alpha[mt * 16 + (lane >> 2)], f1 = s_alpha[mt * 16 + (lane >> 2) + 8];
-#pragma unroll
-      for (int k = 0; k < 4; ++k) al_ldm(smem_u32(s_p) + ((mt * 16 + a_row) * AL_PP + k * 16 + a_col) * 2, pa[mt][k]);
-      if (__any_sync(0xffffffffu, f0 != 1.f || f1 != 1.f)) {
-#pragma unroll
-        for (int i = 0; i < 2 * NU; ++i) { o[mt][i][0] *= f0; o[mt][i][1] *= f0; o[mt][i][2] *= f1; o[mt][i][3] *= f1; }
-      }
-    }
-#pragma unroll
-    for (int u = 0; u < NU; ++u) {
-      const int col = (warp + 8 * u) * 16;
-      if (col < rank) {
-        const uint32_t va = kt + (a_row * KP + col + a_col) * 2;
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          uint32_t vb[4];
-          al_ldm_t(va + k * 16 * KP * 2, vb);
-#pragma unroll
-          for (int mt = 0; mt < MT; ++mt) {
-            al_mma(o[mt][2 * u], pa[mt][k], vb[0], vb[1]);
-            al_mma(o[mt][2 * u + 1], pa[mt][k], vb[2], vb[3]);
+          for (int i = 0; i < N / 4; ++i) {
+            const float4 a = al[i];
+            o[k][4 * i] = o[k][4 * i] * a.x + __uint_as_float(v[4 * i]);
+            o[k][4 * i + 1] = o[k][4 * i + 1] * a.y + __uint_as_float(v[4 * i + 1]);
+            o[k][4 * i + 2] = o[k][4 * i + 2] * a.z + __uint_as_float(v[4 * i + 2]);
+            o[k][4 * i + 3] = o[k][4 * i + 3] * a.w + __uint_as_float(v[4 * i + 3]);
           }
         }
       }
+      tc_fence_before();
+      return true;
+    };
+    const int first_pos = start + g0 / H, key_in_chunk = (qd & 1) * 32 + lane;
+    uint8_t* p_chunk = pP + (qd >> 1) * QCHUNK;
+    // A warp whose wait fails still meets the others at the barriers: every turn has one, whatever happened before.
+    for (int j = 0; j < nt; ++j) {
+      const int turn = j & 1;
+      ok = ok && wait_all(B_SFULL + turn, (j >> 1) & 1u);
+      float v[NC];
+      const int tile0 = (ta + j) * AL_KEYS, key = tile0 + qd * 32 + lane;
+      if (ok) {
+        tc_fence_after();
+        uint32_t raw[NC];
+        if constexpr (NC == 16) tmem_ld_x16(t_lane + turn * N + c0, raw); else tmem_ld_x8(t_lane + turn * N + c0, raw);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < NC; ++i) v[i] = __uint_as_float(raw[i]) * p.scale_log2;
+        if (tile0 + AL_KEYS - 1 > first_pos) {
+#pragma unroll
+          for (int i = 0; i < NC; ++i) if (key > sh.pos[c0 + i]) v[i] = -INFINITY;
+        }
+        float mine = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+          const float m = al_warp_max(v[i]);
+          if (lane == i) mine = m;
+        }
+        if (lane < NC) sh.red[turn][qd][c0 + lane] = mine;
+      }
+      named_bar_sync(1, AL_SOFTMAX);
+      if (!ok) continue;
+      float a_mine = 0.f;
+#pragma unroll
+      for (int i = 0; i < NC; i += 4) {
+        const float4 x0 = *reinterpret_cast<const float4*>(&sh.red[turn][0][c0 + i]), x1 = *reinterpret_cast<const float4*>(&sh.red[turn][1][c0 + i]);
+        const float4 x2 = *reinterpret_cast<const float4*>(&sh.red[turn][2][c0 + i]), x3 = *reinterpret_cast<const float4*>(&sh.red[turn][3][c0 + i]);
+        const float mx[4] = {fmaxf(fmaxf(x0.x, x1.x), fmaxf(x2.x, x3.x)), fmaxf(fmaxf(x0.y, x1.y), fmaxf(x2.y, x3.y)),
+                             fmaxf(fmaxf(x0.z, x1.z), fmaxf(x2.z, x3.z)), fmaxf(fmaxf(x0.w, x1.w), fmaxf(x2.w, x3.w))};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const int c = i + k;
+          const float m_new = fmaxf(m_run[c], mx[k]), m_use = m_new == -INFINITY ? 0.f : m_new;
+          const float alpha = m_run[c] == -INFINITY ? 0.f : exp2f(m_run[c] - m_use);
+          m_run[c] = m_new;
+          if (lane == c) a_mine = alpha;
+          const __nv_bfloat16 e = __float2bfloat16(exp2f(v[c] - m_use));
+          l_run[c] = l_run[c] * alpha + __bfloat162float(e);             // what the MMA will actually see
+          *reinterpret_cast<__nv_bfloat16*>(p_chunk + (p.ahead ? turn * 2 * QCHUNK : 0) + al_swizzled(c0 + c, key_in_chunk)) = e;
+        }
+      }
+      if (qd == 0 && lane < NC) sh.alpha[turn][c0 + lane] = a_mine;
+      tc_fence_before();
+      fence_proxy_async_smem();
+      mbar_arrive(bar(B_PFULL));
+      if (j > 0 && !o_update(j - 1)) ok = false;
     }
-  }
-
+    named_bar_sync(1, AL_SOFTMAX);                       // the last turn's factors are written
+    if (ok && nt > 0) ok = o_update(nt - 1);
 #pragma unroll
-  for (int w = TPR / 2; w > 0; w >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, w);
-  __syncthreads();                                       // the key tiles become the merge buffer
-  float* obuf = reinterpret_cast<float*>(al_smem_raw);
-  const int OP = rank + 4;
+    for (int i = 0; i < NC; ++i) {
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int i = 0; i < 2 * NU; ++i) {
-      const int d = (warp + 8 * (i >> 1)) * 16 + (i & 1) * 8 + (lane & 3) * 2, r = mt * 16 + (lane >> 2);
-      if (d < rank) {
-        *reinterpret_cast<float2*>(obuf + r * OP + d) = make_float2(o[mt][i][0], o[mt][i][1]);
-        *reinterpret_cast<float2*>(obuf + (r + 8) * OP + d) = make_float2(o[mt][i][2], o[mt][i][3]);
+      for (int w = 16; w > 0; w >>= 1) l_run[i] += __shfl_xor_sync(0xffffffffu, l_run[i], w);
+      if (lane == i) {
+        sh.lw[qd][c0 + i] = l_run[i];
+        if (qd == 0) sh.m[c0 + i] = m_run[i];
       }
     }
-  if (my_key == 0) { s_m[my_row] = m_run; s_l[my_row] = l_run; }
+  }
+  tc_fence_before();
+  __syncthreads();                                       // all products are done: the rings become the merge buffer
+  float* obuf = reinterpret_cast<float*>(al_smem);
+  const int OP = rank + 4;
+  if (warp >= 2) {
+    const int half = (warp - 2) >> 2, at = (warp & 3) * 32 + lane;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int dim = (half + 2 * k) * 128 + at;
+      if (dim < rank) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) obuf[i * OP + dim] = o[k][i];
+      }
+    }
+    if (tid - 64 < N) sh.l[tid - 64] = sh.lw[0][tid - 64] + sh.lw[1][tid - 64] + sh.lw[2][tid - 64] + sh.lw[3][tid - 64];
+  } else if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, TMEM_COLS);
+  }
+  __syncwarp();
   if (S > 1) cluster_sync_all(); else __syncthreads();
   if (tid < n_rows) {                                    // the row's factor for every split
-    const uint32_t ma = smem_u32(s_m + tid), la = smem_u32(s_l + tid);
-    float m = -INFINITY, l = 0.f;
-    for (int s = 0; s < S; ++s) m = fmaxf(m, al_ld_cluster(mapa_shared(ma, s)));
-    for (int s = 0; s < S; ++s) {
-      const float ms = al_ld_cluster(mapa_shared(ma, s)), f = ms == -INFINITY ? 0.f : exp2f(ms - m);
-      s_f[s * ROWS + tid] = f;
-      l += f * al_ld_cluster(mapa_shared(la, s));
+    const uint32_t ma = smem_u32(&sh.m[tid]), la = smem_u32(&sh.l[tid]);
+    float ms[8], ls[8], m = -INFINITY, l = 0.f;
+#pragma unroll
+    for (int s = 0; s < 8; ++s) {
+      ms[s] = s < S ? al_ld_cluster(mapa_shared(ma, s)) : -INFINITY;
+      ls[s] = s < S ? al_ld_cluster(mapa_shared(la, s)) : 0.f;
+    }
+#pragma unroll
+    for (int s = 0; s < 8; ++s) m = fmaxf(m, ms[s]);
+#pragma unroll
+    for (int s = 0; s < 8; ++s) {
+      ms[s] = ms[s] == -INFINITY ? 0.f : exp2f(ms[s] - m);
+      l += ms[s] * ls[s];
     }
     const float inv = l > 0.f ? 1.f / l : 0.f;
-    for (int s = 0; s < S; ++s) s_f[s * ROWS + tid] *= inv;
+#pragma unroll
+    for (int s = 0; s < 8; ++s) if (s < S) sh.f[s][tid] = ms[s] * inv;
   }
   __syncthreads();
-  const int half = rank >> 1;
-  for (int i = split * AL_THREADS + tid; i < n_rows * half; i += S * AL_THREADS) {
-    const int r = i / half, d = (i - r * half) * 2, g = g0 + r, tok = g / H;
+  const int quads = rank >> 2;
+  for (int i = split * AL_THREADS + tid; i < n_rows * quads; i += S * AL_THREADS) {
+    const int r = i / quads, d = (i - r * quads) * 4, g = g0 + r, tok = g / H;
     const uint32_t at = smem_u32(obuf + r * OP + d);
-    float v0 = 0.f, v1 = 0.f;
-    for (int s = 0; s < S; ++s) {
-      const uint32_t a = mapa_shared(at, s);
-      const float f = s_f[s * ROWS + r];
-      v0 += f * al_ld_cluster(a);
-      v1 += f * al_ld_cluster(a + 4);
-    }
-    *reinterpret_cast<__nv_bfloat162*>(p.out + static_cast<size_t>(row0 + tok) * p.ldo + static_cast<size_t>(g - tok * H) * rank + d) = __floats2bfloat162_rn(v0, v1);
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int s = 0; s < 8; ++s)
+      if (s < S) {
+        const float f = sh.f[s][r];
+        const float4 x = al_ld_cluster4(mapa_shared(at, s));
+        v.x += f * x.x; v.y += f * x.y; v.z += f * x.z; v.w += f * x.w;
+      }
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p.out + static_cast<size_t>(row0 + tok) * p.ldo + static_cast<size_t>(g - tok * H) * rank + d) =
+        make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
   }
   if (S > 1) cluster_sync_all();                         // no CTA leaves while a peer may still read its partials
 }
 
-template <int MT, int NU>
-static int launch_attn_latent(const AttnLatentParams& p, dim3 grid, cudaStream_t stream) {
+struct AlPlan { int slots, rot_slots, ahead, smem; };
+
+// rings that fit; false: sizes beyond the kernel
+static bool al_plan(int rank, int rot, int n, AlPlan& plan) {
+  if (rank <= 0 || rank > 512 || rot < 0 || rot > 128 || rank % 8 || rot % 8) return false;
+  const int nd = (rank + 127) / 128, kq = (rank + 63) / 64, rc = (rot + 63) / 64;
+  const int tail = n == 16 ? static_cast<int>(sizeof(AlShared<16>)) : static_cast<int>(sizeof(AlShared<32>));
+  auto bytes = [&](int slots, int rs, int ahead) { return slots * AL_SLOT + rs * rc * AL_CHUNK + (kq + rc) * n * 128 + (ahead ? 2 : 1) * 2 * n * 128 + tail; };
+  for (int ahead = 1; ahead >= 0; --ahead)
+    for (int rs = 2; rs >= 1; --rs) {
+      int slots = ahead ? 2 * nd : nd;
+      if (bytes(slots, rs, ahead) > AL_MAX_SMEM) continue;
+      while (slots < AL_MAX_SLOTS && bytes(slots + 1, rs, ahead) <= AL_MAX_SMEM) ++slots;
+      if (!ahead && rs == 2 && slots == nd) continue;      // a spare slot is worth more than a second one for the rotated part
+      plan = {slots, rs, ahead, bytes(slots, rs, ahead)};
+      return n * (rank + 4) * 4 <= slots * AL_SLOT;
+    }
+  return false;
+}
+
+template <int N>
+static int launch_attn_latent(const CUtensorMap& tq, const CUtensorMap& tc, const CUtensorMap& tr, const AttnLatentParams& p, dim3 grid, int smem, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_latent_kernel<MT, NU>, cudaFuncAttributeMaxDynamicSharedMemorySize, AL_MAX_SMEM);
+    cudaError_t e = cudaFuncSetAttribute(attn_latent_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, AL_MAX_SMEM);
     if (e != cudaSuccess) return -1000 - static_cast<int>(e);
-    cudaFuncSetAttribute(attn_latent_kernel<MT, NU>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
     configured = true;
   }
-  launch_ex(attn_latent_kernel<MT, NU>, grid, dim3(AL_THREADS), al_smem(p.d.rank + p.d.rot, MT), stream, p.splits, p);
+  launch_ex(attn_latent_kernel<N>, grid, dim3(AL_THREADS), smem, stream, p.splits, tq, tc, tr, p);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -2000 - static_cast<int>(e);
 }
@@ -314,12 +445,9 @@ bool latent_cache_ok(const b200_paged_cache* c, const b200_latent_dims* d);     
 
 using namespace b200;
 
-// CTAs per SM the kernel reaches with these sizes (16 or 32 rows per CTA); 0: sizes beyond it
-extern "C" int b200_attn_latent_ctas_per_sm(int rank, int rot, int rows) {
-  if (rank <= 0 || rank > 512 || rot < 0 || rank % 8 || rot % 8) return 0;
-  const int smem = al_smem(rank + rot, rows > 16 ? 2 : 1) + 1024, merge = 16 * (rows > 16 ? 2 : 1) * (rank + 4) * 4;
-  if (smem > AL_MAX_SMEM || merge > 2 * AL_KEYS * al_kp(rank + rot) * 2) return 0;
-  return rank <= 256 && 2 * smem <= AL_MAX_SMEM ? 2 : 1;
+extern "C" int b200_attn_latent_fits(int rank, int rot) {
+  AlPlan plan;
+  return al_plan(rank, rot, 16, plan) && al_plan(rank, rot, 32, plan) ? 1 : 0;
 }
 
 extern "C" int b200_attn_latent(const void* q, long long ldq, const void* q_rot, long long ldr, int head_ld_rot, void* out, long long ldo,
@@ -328,19 +456,27 @@ extern "C" int b200_attn_latent(const void* q, long long ldq, const void* q_rot,
                                 const b200_paged_cache* cache, int splits, int* status, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (!q || !q_rot || !out || !positions || !latent_cache_ok(cache, d) || cache->f32 || cache->page_size != AL_PS) return -1;
-  if (ldq % 8 || ldo % 2 || ldr % 2 || head_ld_rot % 2 || (reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(q_rot) & 3)) return -2;
+  if (ldq != static_cast<long long>(d->heads) * d->rank || ldo % 4 || ldr % 2 || head_ld_rot % 2 || (reinterpret_cast<uintptr_t>(q) & 15) ||
+      (reinterpret_cast<uintptr_t>(out) & 7) || (reinterpret_cast<uintptr_t>(q_rot) & 3)) return -2;
   if (splits < 1 || splits > 8 || max_pos <= 0 || (d->true_rot > 0 && (!cos_tab || !sin_tab)) || (cu && (portions <= 0 || max_len <= 0))) return -3;
   const int longest = cu ? max_len : 1, batch = cu ? portions : M;
-  const int mt = static_cast<long long>(longest) * d->heads > 16 ? 2 : 1;
-  if (b200_attn_latent_ctas_per_sm(d->rank, d->rot, 16 * mt) == 0) return -4;
-  AttnLatentParams p;
-  p.q = static_cast<const __nv_bfloat16*>(q); p.ldq = ldq; p.q_rot = static_cast<const __nv_bfloat16*>(q_rot); p.ldr = ldr; p.head_ld_rot = head_ld_rot;
-  p.out = static_cast<__nv_bfloat16*>(out); p.ldo = ldo; p.d = *d; p.scale_log2 = scale * AL_LOG2E; p.cu = cu; p.positions = positions;
-  p.seq_ids = seq_ids; p.seq_lens = seq_lens; p.cos_tab = cos_tab; p.sin_tab = sin_tab; p.max_pos = max_pos; p.splits = splits; p.c = *cache; p.status = status;
-  const long long tiles = (static_cast<long long>(longest) * d->heads + 16 * mt - 1) / (16 * mt);
+  const int n = static_cast<long long>(longest) * d->heads > 16 ? 32 : 16;
+  AlPlan plan;
+  if (!al_plan(d->rank, d->rot, n, plan)) return -4;
+  const long long tiles = (static_cast<long long>(longest) * d->heads + n - 1) / n;
   if (tiles > 65535 || batch > 65535) return -5;
+  const int dk = d->rank + d->rot;
+  const uint64_t rows = static_cast<uint64_t>(M) * d->heads, pitch = static_cast<uint64_t>(dk) * 2;
+  CUtensorMap tq, tc, tr;
+  if (make_tmap_3d_bf16(&tq, q, d->rank, rows, 1, static_cast<uint64_t>(d->rank) * 2, rows * d->rank * 2, n, 1)) return -11;
+  if (make_tmap_3d_bf16(&tc, cache->data, d->rank, AL_PS, cache->num_pages, pitch, pitch * AL_PS, AL_PS, 1)) return -12;
+  tr = tc;
+  if (d->rot > 0 && make_tmap_3d_bf16(&tr, static_cast<const uint8_t*>(cache->data) + static_cast<size_t>(d->rank) * 2, d->rot, AL_PS, cache->num_pages, pitch, pitch * AL_PS, AL_PS, 1)) return -13;
+  AttnLatentParams p;
+  p.q_rot = static_cast<const __nv_bfloat16*>(q_rot); p.ldr = ldr; p.head_ld_rot = head_ld_rot;
+  p.out = static_cast<__nv_bfloat16*>(out); p.ldo = ldo; p.d = *d; p.scale_log2 = scale * AL_LOG2E; p.cu = cu; p.positions = positions;
+  p.seq_ids = seq_ids; p.seq_lens = seq_lens; p.cos_tab = cos_tab; p.sin_tab = sin_tab; p.max_pos = max_pos; p.splits = splits;
+  p.slots = plan.slots; p.rot_slots = plan.rot_slots; p.ahead = plan.ahead; p.c = *cache; p.status = status; p.limit_ns = 2000000000ull;
   const dim3 grid(splits, static_cast<unsigned>(tiles), batch);
-  const int nu = d->rank <= 128 ? 1 : (d->rank <= 256 ? 2 : 4);
-  if (mt == 1) return nu == 1 ? launch_attn_latent<1, 1>(p, grid, stream) : (nu == 2 ? launch_attn_latent<1, 2>(p, grid, stream) : launch_attn_latent<1, 4>(p, grid, stream));
-  return nu == 1 ? launch_attn_latent<2, 1>(p, grid, stream) : (nu == 2 ? launch_attn_latent<2, 2>(p, grid, stream) : launch_attn_latent<2, 4>(p, grid, stream));
+  return n == 16 ? launch_attn_latent<16>(tq, tc, tr, p, grid, plan.smem, stream) : launch_attn_latent<32>(tq, tc, tr, p, grid, plan.smem, stream);
 }

@@ -113,7 +113,7 @@ class _Sig:
     b200_rotary_heads = (I, [P, LL, I, I, I, I, I, I, P, P, P, I, P, P])
     b200_latent_gather = (I, [P, P, P, I, I, P, P, P])
     b200_attn_latent_any = (I, [P, LL, P, LL, I, P, LL, I, P, F, P, P, P, P, P, P])
-    b200_attn_latent_ctas_per_sm = (I, [I, I, I])
+    b200_attn_latent_fits = (I, [I, I])
     b200_attn_latent = (I, [P, LL, P, LL, I, P, LL, I, P, F, P, I, I, P, P, P, P, P, I, P, I, P, P])
     b200_attn_prefill_latent_fits = (I, [I, I, I])
     b200_attn_prefill_latent = (I, [P, LL, I, I, I, I, P, LL, P, LL, I, P, LL, I, I, I, F, P, P, P, P, LL, P, P])

@@ -65,18 +65,15 @@ def attend_any(q: torch.Tensor, q_rot: torch.Tensor, rot_head_ld: int, dm, scale
     return out
 
 
-def fits(dm, dtype: torch.dtype, page_size: int, rows_per_portion: int = 32) -> bool:
+def fits(dm, dtype: torch.dtype, page_size: int) -> bool:
     """Whether ``attend`` takes these sizes (``attend_any`` takes all)."""
-    return (dtype == torch.bfloat16 and page_size == PAGE and
-            _lib.lib().b200_attn_latent_ctas_per_sm(dm.rank, dm.rot, rows_per_portion) > 0)
+    return dtype == torch.bfloat16 and page_size == PAGE and bool(_lib.lib().b200_attn_latent_fits(dm.rank, dm.rot))
 
 
 def pick_splits(batch: int, row_tiles: int, keys: int, slots: int) -> int:
-    """CTAs per row tile: as many as still make one wave, with at least two tiles of 64 keys each."""
-    pairs, s = max(1, batch * row_tiles), 1
-    while s < 8 and pairs * s * 2 <= slots and keys // (2 * s) >= 128:
-        s *= 2
-    return s
+    """CTAs per row tile: as many as still make one wave, with at least one tile of 128 keys each."""
+    pairs = max(1, batch * row_tiles)
+    return max(1, min(8, slots // pairs, keys // 128))
 
 
 def attend(q: torch.Tensor, q_raw: torch.Tensor, raw_head_ld: int, dm, scale: float, positions: torch.Tensor, seq_ids: torch.Tensor | None,
@@ -90,8 +87,7 @@ def attend(q: torch.Tensor, q_raw: torch.Tensor, raw_head_ld: int, dm, scale: fl
     if splits is None:
         longest, batch = (int(max_len), cu.numel() - 1) if cu is not None else (1, M)
         per_cta = 32 if longest * dm.heads > 16 else 16
-        slots = _lib.num_sms(q.device.index) * _lib.lib().b200_attn_latent_ctas_per_sm(dm.rank, dm.rot, per_cta)
-        splits = pick_splits(batch, -(-longest * dm.heads // per_cta), keys or page_table.shape[1] * cache.page_size, slots)
+        splits = pick_splits(batch, -(-longest * dm.heads // per_cta), keys or page_table.shape[1] * cache.page_size, _lib.num_sms(q.device.index))
     _lib.check(_lib.lib().b200_attn_latent(
         q.data_ptr(), q.stride(0), q_raw.data_ptr(), q_raw.stride(0), raw_head_ld, out.data_ptr(), out.stride(0), M, ctypes.byref(dm),
         float(scale), _lib.ptr(cu), cu.numel() - 1 if cu is not None else 0, int(max_len), positions.data_ptr(), _lib.ptr(seq_ids),
