@@ -3,11 +3,12 @@
 // `rank` dimensions are also its value, so a cached row is fetched once, by TMA, and serves both products from shared memory.
 //
 // Rows are (token, head) pairs of one portion in order, N = 16 or 32 of them per CTA.  So few rows would waste the MMA's 128, so
-// the keys take that side:  S^T [128 keys, N] = C [128, dk] . Q^T,   O^T [rank, N] = C^T [rank, 128] . P^T in blocks of 128 value
-// dimensions - the same operand tile, once K-major and once MN-major.
-//   warp 0      TMA producer: a tile is 128 keys = 8 pages, in slots of 128 latent columns and one of the rotated part, each
-//               released as soon as its last product is done (rings; a tile of 512 + 64 columns is 144 KB, so the next one
-//               streams in as this one leaves).  In decoding the tiles of earlier tokens are requested before the dependency
+// the keys take that side:  S^T [keys, N] = C [keys, dk] . Q^T,   O^T [rank, N] = C^T [rank, keys] . P^T in blocks of 128 value
+// dimensions - the same operand tile, once K-major and once MN-major.  Tiles are 128 keys (512 + 64 columns x 128 keys are
+// 144 KB) where the queries leave room for one, else 64: the score MMA then still has 128 rows, and the upper half, whatever lies
+// behind the operand, is never read back.
+//   warp 0      TMA producer: a tile is 8 or 4 pages, in slots of 128 latent columns and one of the rotated part, each
+//               released as soon as its last product is done (rings).  In decoding the tiles of earlier tokens are requested before the dependency
 //               wait: only the new token's row is written by a kernel that may still run.
 //   warp 1      MMA issuer; where two tiles fit, the scores of the next tile go before the values of this one
 //   warps 2..9  softmax with keys on the lanes: a warp holds 32 keys of half the rows; maxima by warp reduction and through
@@ -21,10 +22,8 @@
 
 namespace b200 {
 
-constexpr int AL_THREADS = 320, AL_SOFTMAX = 256, AL_KEYS = 128, AL_PS = 16;
-constexpr int AL_CHUNK = 128 * 128;                  // 128 keys x 64 bf16
-constexpr int AL_SLOT = 2 * AL_CHUNK;                // 128 latent columns
-constexpr int AL_MAX_SMEM = 232448, AL_MAX_SLOTS = 8;
+constexpr int AL_THREADS = 320, AL_SOFTMAX = 256, AL_PS = 16;
+constexpr int AL_MAX_SMEM = 232448, AL_MAX_SLOTS = 12, AL_MAX_ROT = 3;
 constexpr float AL_LOG2E = 1.4426950408889634f;
 
 struct AttnLatentParams {
@@ -67,16 +66,18 @@ struct AlShared {      // behind the operands
   float m[N], l[N], lw[4][N];
   float f[8][N];       // factor of every split
   int pos[N];
-  uint64_t bars[2 * AL_MAX_SLOTS + 16];
+  uint64_t bars[2 * AL_MAX_SLOTS + 2 * AL_MAX_ROT + 8];
   uint32_t tmem;
   int abort;
 };
 
-template <int N>
+template <int N, int KEYS>
 __global__ void __launch_bounds__(AL_THREADS, 1)
 attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_c,
                    const __grid_constant__ CUtensorMap tmap_r, const __grid_constant__ AttnLatentParams p) {
   constexpr int NC = N / 2;                              // columns of a softmax thread
+  constexpr int AL_KEYS = KEYS, AL_CHUNK = KEYS * 128, AL_SLOT = 2 * AL_CHUNK, PAGES = KEYS / AL_PS;      // chunk: 64 bf16 of every key
+  constexpr int PCHUNKS = KEYS / 64;                     // 64-key chunks of the softmax weights
   constexpr int QCHUNK = N * 128, TMEM_COLS = N == 32 ? 512 : 256, TMEM_O = 2 * N;
   pdl_launch_dependents();
   if (p.cu) pdl_wait();                                  // decoding: page table, positions and earlier rows are older than this step
@@ -105,9 +106,10 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   const uint32_t sC = smem_u32(al_smem), sR = sC + p.slots * AL_SLOT, sQ = sR + p.rot_slots * rc * AL_CHUNK, sP = sQ + (kq + rc) * QCHUNK;
   uint8_t* pQr = al_smem + (sQ - sC) + kq * QCHUNK;
   uint8_t* pP = al_smem + (sP - sC);
-  AlShared<N>& sh = *reinterpret_cast<AlShared<N>*>(pP + (p.ahead ? 2 : 1) * 2 * QCHUNK);
+  AlShared<N>& sh = *reinterpret_cast<AlShared<N>*>(pP + (p.ahead ? 2 : 1) * PCHUNKS * QCHUNK);
   const uint32_t bar0 = smem_u32(sh.bars);
-  enum { B_Q = 0, B_QROT = 1, B_SFULL = 2, B_PFULL = 4, B_OFULL = 5, B_RFULL = 7, B_REMPTY = 9, B_CFULL = 11, B_CEMPTY = 11 + AL_MAX_SLOTS, B_COUNT = 11 + 2 * AL_MAX_SLOTS };
+  enum { B_Q = 0, B_QROT = 1, B_SFULL = 2, B_PFULL = 4, B_OFULL = 5, B_RFULL = 7, B_REMPTY = 7 + AL_MAX_ROT, B_CFULL = 7 + 2 * AL_MAX_ROT,
+         B_CEMPTY = B_CFULL + AL_MAX_SLOTS, B_COUNT = B_CEMPTY + AL_MAX_SLOTS };
   auto bar = [&](int i) { return bar0 + 8u * i; };
   volatile int* abort_flag = &sh.abort;
   const uint64_t limit = p.limit_ns;
@@ -134,7 +136,7 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   if (warp == 0) {
     const int* pt = p.c.page_table + static_cast<size_t>(seq) * p.c.max_pages;
     auto page_of = [&](int t) {                          // lane <-> page of tile t; past the last key: out of range, arrives as zeros
-      const int tok = t * AL_KEYS + (lane & 7) * AL_PS;
+      const int tok = t * AL_KEYS + (lane % PAGES) * AL_PS;
       const int pg = tok <= last_pos ? pt[tok / AL_PS] : p.c.num_pages;
       return pg < 0 || pg > p.c.num_pages ? p.c.num_pages : pg;
     };
@@ -152,9 +154,9 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         if (!ok) break;
         if (lane == 0) mbar_expect_tx(bar(B_CFULL + cs), chunks * AL_CHUNK);
         __syncwarp();
-        // lanes 0..7 fetch the first chunk's pages, 8..15 the second's
-        if (lane < 8 * chunks)
-          tma_load_3d(sC + cs * AL_SLOT + (lane >> 3) * AL_CHUNK + (lane & 7) * 2048, &tmap_c, bar(B_CFULL + cs), (2 * d + (lane >> 3)) * 64, 0, page);
+        // the first lanes fetch the first chunk's pages, the next ones the second's
+        if (lane < PAGES * chunks)
+          tma_load_3d(sC + cs * AL_SLOT + (lane / PAGES) * AL_CHUNK + (lane % PAGES) * 2048, &tmap_c, bar(B_CFULL + cs), (2 * d + lane / PAGES) * 64, 0, page);
         if (++cs == p.slots) { cs = 0; cp ^= 1u; }
       }
       if (ok && rc > 0) {
@@ -162,8 +164,8 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         if (!ok) break;
         if (lane == 0) mbar_expect_tx(bar(B_RFULL + rs), rc * AL_CHUNK);
         __syncwarp();
-        if (lane < 8 * rc)
-          tma_load_3d(sR + rs * rc * AL_CHUNK + (lane >> 3) * AL_CHUNK + (lane & 7) * 2048, &tmap_r, bar(B_RFULL + rs), (lane >> 3) * 64, 0, page);
+        if (lane < PAGES * rc)
+          tma_load_3d(sR + rs * rc * AL_CHUNK + (lane / PAGES) * AL_CHUNK + (lane % PAGES) * 2048, &tmap_r, bar(B_RFULL + rs), (lane / PAGES) * 64, 0, page);
         if (++rs == p.rot_slots) { rs = 0; rp ^= 1u; }
       }
       page = next;
@@ -180,24 +182,32 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       const int c_steps = (rank + 15) >> 4, r_steps = (rot + 15) >> 4;
       int cs = 0, rs = 0, vs = 0;                        // slots: scores read cs, values vs
       uint32_t cp = 0, rp = 0;
+      // One thread issues everything, so a descriptor must cost an addition: bases here, offsets known at compile time below
+      // (the address field counts 16 bytes).
+      const uint64_t c_desc = umma_desc_k_sw128(sC), ct_desc = umma_desc_mn_sw128(sC, AL_CHUNK, 1024), r_desc = umma_desc_k_sw128(sR),
+                     q_desc = umma_desc_k_sw128(sQ), qr_desc = umma_desc_k_sw128(sQ + kq * QCHUNK), p_desc = umma_desc_k_sw128(sP);
       auto issue_s = [&](int j) -> bool {
         const uint32_t d_tmem = tmem_base + (j & 1) * N;
-        uint32_t acc = 0;
         for (int d = 0; d < nd; ++d) {
           if (!mbar_wait(bar(B_CFULL + cs), cp, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (18 << 8)), limit)) return false;
           tc_fence_after();
-          const int steps = min(8, c_steps - 8 * d);
-          for (int kk = 0; kk < steps; ++kk, acc = 1)
-            umma_f16_ss(d_tmem, umma_desc_k_sw128(sC + cs * AL_SLOT + (kk >> 2) * AL_CHUNK) + 2ull * (kk & 3),
-                        umma_desc_k_sw128(sQ + (2 * d + (kk >> 2)) * QCHUNK) + 2ull * (kk & 3), IDESC_S, acc);
+          const int steps = c_steps - 8 * d;
+          const uint64_t a = c_desc + static_cast<uint32_t>(cs * (AL_SLOT >> 4)), bq = q_desc + static_cast<uint32_t>(d * (2 * QCHUNK >> 4));
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk)
+            if (kk < steps)
+              umma_f16_ss(d_tmem, a + ((kk >> 2) * (AL_CHUNK >> 4) + 2 * (kk & 3)), bq + ((kk >> 2) * (QCHUNK >> 4) + 2 * (kk & 3)), IDESC_S,
+                          kk > 0 ? 1u : (d > 0 ? 1u : 0u));
           if (++cs == p.slots) { cs = 0; cp ^= 1u; }
         }
         if (rc > 0) {
           if (!mbar_wait(bar(B_RFULL + rs), rp, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (18 << 8)), limit)) return false;
           tc_fence_after();
-          for (int kk = 0; kk < r_steps; ++kk, acc = 1)
-            umma_f16_ss(d_tmem, umma_desc_k_sw128(sR + (rs * rc + (kk >> 2)) * AL_CHUNK) + 2ull * (kk & 3),
-                        umma_desc_k_sw128(sQ + (kq + (kk >> 2)) * QCHUNK) + 2ull * (kk & 3), IDESC_S, acc);
+          const uint64_t a = r_desc + static_cast<uint32_t>(rs * rc * (AL_CHUNK >> 4));
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk)
+            if (kk < r_steps)
+              umma_f16_ss(d_tmem, a + ((kk >> 2) * (AL_CHUNK >> 4) + 2 * (kk & 3)), qr_desc + ((kk >> 2) * (QCHUNK >> 4) + 2 * (kk & 3)), IDESC_S, 1u);
           umma_commit(bar(B_REMPTY + rs));
           if (++rs == p.rot_slots) { rs = 0; rp ^= 1u; }
         }
@@ -211,13 +221,13 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         if (p.ahead && j + 1 < nt && !issue_s(j + 1)) { ok = false; break; }
         if (!mbar_wait(bar(B_PFULL), j & 1u, abort_flag, p.status, (ST_TIMEOUT_PEER_FLAG | (18 << 8)), limit)) { ok = false; break; }
         tc_fence_after();
-        const uint32_t pd = sP + (p.ahead ? (j & 1) * 2 * QCHUNK : 0);
+        const uint64_t bp = p_desc + (p.ahead ? static_cast<uint32_t>((j & 1) * (PCHUNKS * QCHUNK >> 4)) : 0u);
         for (int d = 0; d < nd; ++d) {
           const uint32_t d_tmem = tmem_base + TMEM_O + ((j & 1) * 4 + d) * N;
+          const uint64_t a = ct_desc + static_cast<uint32_t>(vs * (AL_SLOT >> 4));
 #pragma unroll
-          for (int kk = 0; kk < 8; ++kk)
-            umma_f16_ss(d_tmem, umma_desc_mn_sw128(sC + vs * AL_SLOT + kk * 2048, AL_CHUNK, 1024),
-                        umma_desc_k_sw128(pd + (kk >> 2) * QCHUNK) + 2ull * (kk & 3), IDESC_O, kk > 0 ? 1u : 0u);
+          for (int kk = 0; kk < KEYS / 16; ++kk)
+            umma_f16_ss(d_tmem, a + kk * (2048 >> 4), bp + ((kk >> 2) * (QCHUNK >> 4) + 2 * (kk & 3)), IDESC_O, kk > 0 ? 1u : 0u);
           umma_commit(bar(B_CEMPTY + vs));
           if (++vs == p.slots) vs = 0;
         }
@@ -288,8 +298,9 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       ok = ok && wait_all(B_SFULL + turn, (j >> 1) & 1u);
       float v[NC];
       const int tile0 = (ta + j) * AL_KEYS, key = tile0 + qd * 32 + lane;
-      if (ok) {
-        tc_fence_after();
+      if (ok) tc_fence_after();
+      const bool mine_here = qd < KEYS / 32;             // the upper lanes of a 64-key tile hold nothing
+      if (ok && mine_here) {
         uint32_t raw[NC];
         if constexpr (NC == 16) tmem_ld_x16(t_lane + turn * N + c0, raw); else tmem_ld_x8(t_lane + turn * N + c0, raw);
         tmem_ld_wait();
@@ -312,10 +323,12 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       float a_mine = 0.f;
 #pragma unroll
       for (int i = 0; i < NC; i += 4) {
-        const float4 x0 = *reinterpret_cast<const float4*>(&sh.red[turn][0][c0 + i]), x1 = *reinterpret_cast<const float4*>(&sh.red[turn][1][c0 + i]);
-        const float4 x2 = *reinterpret_cast<const float4*>(&sh.red[turn][2][c0 + i]), x3 = *reinterpret_cast<const float4*>(&sh.red[turn][3][c0 + i]);
-        const float mx[4] = {fmaxf(fmaxf(x0.x, x1.x), fmaxf(x2.x, x3.x)), fmaxf(fmaxf(x0.y, x1.y), fmaxf(x2.y, x3.y)),
-                             fmaxf(fmaxf(x0.z, x1.z), fmaxf(x2.z, x3.z)), fmaxf(fmaxf(x0.w, x1.w), fmaxf(x2.w, x3.w))};
+        float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+        for (int q = 0; q < KEYS / 32; ++q) {
+          const float4 x = *reinterpret_cast<const float4*>(&sh.red[turn][q][c0 + i]);
+          mx[0] = fmaxf(mx[0], x.x); mx[1] = fmaxf(mx[1], x.y); mx[2] = fmaxf(mx[2], x.z); mx[3] = fmaxf(mx[3], x.w);
+        }
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
           const int c = i + k;
@@ -323,9 +336,11 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
           const float alpha = m_run[c] == -INFINITY ? 0.f : exp2f(m_run[c] - m_use);
           m_run[c] = m_new;
           if (lane == c) a_mine = alpha;
-          const __nv_bfloat16 e = __float2bfloat16(exp2f(v[c] - m_use));
-          l_run[c] = l_run[c] * alpha + __bfloat162float(e);             // what the MMA will actually see
-          *reinterpret_cast<__nv_bfloat16*>(p_chunk + (p.ahead ? turn * 2 * QCHUNK : 0) + al_swizzled(c0 + c, key_in_chunk)) = e;
+          if (mine_here) {
+            const __nv_bfloat16 e = __float2bfloat16(exp2f(v[c] - m_use));
+            l_run[c] = l_run[c] * alpha + __bfloat162float(e);           // what the MMA will actually see
+            *reinterpret_cast<__nv_bfloat16*>(p_chunk + (p.ahead ? turn * PCHUNKS * QCHUNK : 0) + al_swizzled(c0 + c, key_in_chunk)) = e;
+          }
         }
       }
       if (qd == 0 && lane < NC) sh.alpha[turn][c0 + lane] = a_mine;
@@ -406,35 +421,40 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   if (S > 1) cluster_sync_all();                         // no CTA leaves while a peer may still read its partials
 }
 
-struct AlPlan { int slots, rot_slots, ahead, smem; };
+struct AlPlan { int keys, slots, rot_slots, ahead, smem; };
 
-// rings that fit; false: sizes beyond the kernel
+// tile and rings that fit; false: sizes beyond the kernel
 static bool al_plan(int rank, int rot, int n, AlPlan& plan) {
   if (rank <= 0 || rank > 512 || rot < 0 || rot > 128 || rank % 8 || rot % 8) return false;
   const int nd = (rank + 127) / 128, kq = (rank + 63) / 64, rc = (rot + 63) / 64;
   const int tail = n == 16 ? static_cast<int>(sizeof(AlShared<16>)) : static_cast<int>(sizeof(AlShared<32>));
-  auto bytes = [&](int slots, int rs, int ahead) { return slots * AL_SLOT + rs * rc * AL_CHUNK + (kq + rc) * n * 128 + (ahead ? 2 : 1) * 2 * n * 128 + tail; };
-  for (int ahead = 1; ahead >= 0; --ahead)
-    for (int rs = 2; rs >= 1; --rs) {
-      int slots = ahead ? 2 * nd : nd;
-      if (bytes(slots, rs, ahead) > AL_MAX_SMEM) continue;
-      while (slots < AL_MAX_SLOTS && bytes(slots + 1, rs, ahead) <= AL_MAX_SMEM) ++slots;
-      if (!ahead && rs == 2 && slots == nd) continue;      // a spare slot is worth more than a second one for the rotated part
-      plan = {slots, rs, ahead, bytes(slots, rs, ahead)};
-      return n * (rank + 4) * 4 <= slots * AL_SLOT;
+  for (int keys = 128; keys >= 64; keys /= 2)
+    for (int ahead = 1; ahead >= 0; --ahead) {
+      auto bytes = [&](int slots, int rs) { return slots * keys * 256 + rs * rc * keys * 128 + (kq + rc) * n * 128 + (ahead ? 2 : 1) * (keys / 64) * n * 128 + tail; };
+      int slots = ahead ? 2 * nd : nd, rs = 1;
+      if (bytes(slots, rs) > AL_MAX_SMEM) continue;
+      // a third tile of the rotated part only beside a third tile of latents
+      while (true) {
+        if (rs < 2 && bytes(slots, rs + 1) <= AL_MAX_SMEM) ++rs;
+        else if (slots < AL_MAX_SLOTS && bytes(slots + 1, rs) <= AL_MAX_SMEM) ++slots;
+        else if (rs < AL_MAX_ROT && slots >= 3 * nd && bytes(slots, rs + 1) <= AL_MAX_SMEM) ++rs;
+        else break;
+      }
+      plan = {keys, slots, rs, ahead, bytes(slots, rs)};
+      return n * (rank + 4) * 4 <= slots * keys * 256;
     }
   return false;
 }
 
-template <int N>
+template <int N, int KEYS>
 static int launch_attn_latent(const CUtensorMap& tq, const CUtensorMap& tc, const CUtensorMap& tr, const AttnLatentParams& p, dim3 grid, int smem, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_latent_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, AL_MAX_SMEM);
+    cudaError_t e = cudaFuncSetAttribute(attn_latent_kernel<N, KEYS>, cudaFuncAttributeMaxDynamicSharedMemorySize, AL_MAX_SMEM);
     if (e != cudaSuccess) return -1000 - static_cast<int>(e);
     configured = true;
   }
-  launch_ex(attn_latent_kernel<N>, grid, dim3(AL_THREADS), smem, stream, p.splits, tq, tc, tr, p);
+  launch_ex(attn_latent_kernel<N, KEYS>, grid, dim3(AL_THREADS), smem, stream, p.splits, tq, tc, tr, p);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -2000 - static_cast<int>(e);
 }
@@ -478,5 +498,6 @@ extern "C" int b200_attn_latent(const void* q, long long ldq, const void* q_rot,
   p.seq_ids = seq_ids; p.seq_lens = seq_lens; p.cos_tab = cos_tab; p.sin_tab = sin_tab; p.max_pos = max_pos; p.splits = splits;
   p.slots = plan.slots; p.rot_slots = plan.rot_slots; p.ahead = plan.ahead; p.c = *cache; p.status = status; p.limit_ns = 2000000000ull;
   const dim3 grid(splits, static_cast<unsigned>(tiles), batch);
-  return n == 16 ? launch_attn_latent<16>(tq, tc, tr, p, grid, plan.smem, stream) : launch_attn_latent<32>(tq, tc, tr, p, grid, plan.smem, stream);
+  if (plan.keys == 128) return n == 16 ? launch_attn_latent<16, 128>(tq, tc, tr, p, grid, plan.smem, stream) : launch_attn_latent<32, 128>(tq, tc, tr, p, grid, plan.smem, stream);
+  return n == 16 ? launch_attn_latent<16, 64>(tq, tc, tr, p, grid, plan.smem, stream) : launch_attn_latent<32, 64>(tq, tc, tr, p, grid, plan.smem, stream);
 }

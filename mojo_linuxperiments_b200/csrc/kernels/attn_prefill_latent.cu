@@ -114,17 +114,18 @@ attn_prefill_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       const int n_steps = (p.dn + 15) >> 4, r_steps = (p.dr + 15) >> 4;
       int ks = 0, vs = 0;
       uint32_t kp = 0, vp = 0;
+      // one thread issues everything: a descriptor costs an addition (the address field counts 16 bytes)
+      const uint64_t q_desc = umma_desc_k_sw128(sQ), k_desc = umma_desc_k_sw128(sK), p_desc = umma_desc_k_sw128(sP), v_desc = umma_desc_mn_sw128(sV, PL_CHUNK, 1024);
       auto issue_s = [&](int j) {                                        // the K stage has been waited for
-        const uint32_t d = tmem_base + (j & 1) * 128, kd = sK + ks * k_bytes;
-        uint32_t acc = 0;
-        auto part = [&](int chunk0, int steps) {
-          for (int kk = 0; kk < steps; ++kk, acc = 1) {
-            const uint32_t off = (chunk0 + (kk >> 2)) * PL_CHUNK;
-            umma_f16_ss(d, umma_desc_k_sw128(sQ + off) + 2ull * (kk & 3), umma_desc_k_sw128(kd + off) + 2ull * (kk & 3), IDESC_S, acc);
-          }
-        };
-        part(0, n_steps);
-        part(nc, r_steps);
+        const uint32_t d = tmem_base + (j & 1) * 128;
+        const uint64_t kd = k_desc + static_cast<uint32_t>(ks * (k_bytes >> 4));
+        for (int c = 0; c < kc; ++c) {
+          const int steps = c < nc ? n_steps - 4 * c : r_steps - 4 * (c - nc);
+          const uint32_t off = c * (PL_CHUNK >> 4);
+#pragma unroll
+          for (int kk = 0; kk < 4; ++kk)
+            if (kk < steps) umma_f16_ss(d, q_desc + (off + 2 * kk), kd + (off + 2 * kk), IDESC_S, kk > 0 ? 1u : (c > 0 ? 1u : 0u));
+        }
         umma_commit(bar(B_KEMPTY + ks));
         umma_commit(bar(B_SFULL + (j & 1)));
         if (++ks == p.k_stages) { ks = 0; kp ^= 1u; }
@@ -141,12 +142,11 @@ attn_prefill_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
         if (!mbar_wait(bar(B_PFULL), j & 1u, abort_flag, p.status, (ST_TIMEOUT_PEER_FLAG | (19 << 8)), limit)) { ok = false; break; }
         if (!mbar_wait(bar(B_VFULL + vs), vp, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (19 << 8)), limit)) { ok = false; break; }
         tc_fence_after();
-        const uint32_t d = tmem_base + 256 + (j & 1) * 128, pd = sP + (p.p_stages == 2 ? (j & 1) * 2 * PL_CHUNK : 0), vd = sV + vs * v_bytes;
+        const uint32_t d = tmem_base + 256 + (j & 1) * 128;
+        const uint64_t a = p_desc + (p.p_stages == 2 ? static_cast<uint32_t>((j & 1) * (2 * PL_CHUNK >> 4)) : 0u), bv = v_desc + static_cast<uint32_t>(vs * (v_bytes >> 4));
 #pragma unroll
-        for (int kk = 0; kk < 8; ++kk) {
-          const uint64_t a = umma_desc_k_sw128(pd + (kk >> 2) * PL_CHUNK) + 2ull * (kk & 3);
-          umma_f16_ss(d, a, umma_desc_mn_sw128(vd + kk * 2048, PL_CHUNK, 1024), idesc_pv, kk > 0 ? 1u : 0u);
-        }
+        for (int kk = 0; kk < 8; ++kk)
+          umma_f16_ss(d, a + ((kk >> 2) * (PL_CHUNK >> 4) + 2 * (kk & 3)), bv + kk * (2048 >> 4), idesc_pv, kk > 0 ? 1u : 0u);
         umma_commit(bar(B_VEMPTY + vs));
         umma_commit(bar(B_OFULL + (j & 1)));
         if (++vs == p.v_stages) { vs = 0; vp ^= 1u; }

@@ -145,7 +145,9 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
     const int q = warp & 3;                 // TMEM lane quarter this warp may read
     float* piece = stage_f + (warp - 2) * 32 * BG_SP;
     int idx = 0;
-    const bool residual = p.epi.mode == B200_EPI_RESIDUAL;
+    const bool residual = p.epi.mode == B200_EPI_RESIDUAL, plain = p.epi.mode == B200_EPI_STORE && !p.epi.gate;
+    const bool plain16 = plain && !p.epi.out_f32, relu2 = p.epi.act == B200_ACT_RELU2;
+    const int r8 = lane >> 2, c8 = (lane & 3) * 8;           // the same with eight columns per lane
     const int rr0 = lane >> 3, c4 = (lane & 7) * 4;          // row group and column quad of this lane in a 32 x 32 piece
     for (int tile = blockIdx.x; tile < num_tiles; tile += gridDim.x, ++idx) {
       const int a = idx & 1;
@@ -187,7 +189,44 @@ bf16_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
                                                                  __uint_as_float(r[4 * g + 2]), __uint_as_float(r[4 * g + 3]));
         __syncwarp();
         const int n = n0 + c * 32 + c4;
-        if (n < p.N) {
+        if (plain16) {
+          const int n8 = n0 + c * 32 + c8;
+          if (n8 < p.N) {
+            __nv_bfloat16* y = static_cast<__nv_bfloat16*>(p.epi.y) + static_cast<long long>(m0 + r8) * p.epi.ldy + n8;
+#pragma unroll
+            for (int it = 0; it < 4; ++it) {
+              const float* src = piece + (it * 8 + r8) * BG_SP + c8;
+              float v[8];
+              *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(src);
+              *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(src + 4);
+              if (relu2) {
+#pragma unroll
+                for (int k = 0; k < 8; ++k) { v[k] = fmaxf(v[k], 0.f); v[k] *= v[k]; }
+              }
+              uint4 o;
+              uint32_t* ow = reinterpret_cast<uint32_t*>(&o);
+#pragma unroll
+              for (int k = 0; k < 4; ++k) {
+                const __nv_bfloat162 pb = __floats2bfloat162_rn(v[2 * k], v[2 * k + 1]);
+                ow[k] = *reinterpret_cast<const uint32_t*>(&pb);
+              }
+              if (m0 + it * 8 + r8 < t.m_end) *reinterpret_cast<uint4*>(y + static_cast<long long>(it * 8) * p.epi.ldy) = o;
+            }
+          }
+        } else if (plain) {
+          if (n < p.N) {
+            float* y = static_cast<float*>(p.epi.y) + static_cast<long long>(m0 + rr0) * p.epi.ldy + n;
+#pragma unroll
+            for (int it = 0; it < 8; ++it) {
+              float4 v = *reinterpret_cast<const float4*>(piece + (it * 4 + rr0) * BG_SP + c4);
+              if (relu2) {
+                v.x = fmaxf(v.x, 0.f); v.y = fmaxf(v.y, 0.f); v.z = fmaxf(v.z, 0.f); v.w = fmaxf(v.w, 0.f);
+                v.x *= v.x; v.y *= v.y; v.z *= v.z; v.w *= v.w;
+              }
+              if (m0 + it * 4 + rr0 < t.m_end) *reinterpret_cast<float4*>(y + static_cast<long long>(it * 4) * p.epi.ldy) = v;
+            }
+          }
+        } else if (n < p.N) {
           if (residual) {
             const EpiNorm nw = epi_norm_columns(p.epi, n);
 #pragma unroll

@@ -14,7 +14,7 @@ template <typename T> __device__ __forceinline__ float la_f(T v);
 template <> __device__ __forceinline__ float la_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ float la_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
 
-constexpr int LA_THREADS = 128;
+constexpr int LA_THREADS = 256;
 
 struct LatentAppendParams {
   const float* in; long long ld;

@@ -12,14 +12,12 @@ namespace b200 {
 
 constexpr int RG_WARPS = 4;
 
-// (value, index) of the warp's largest value; the lowest index wins ties
-__device__ __forceinline__ void rg_argmax(float& v, int& i) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
-    if (ov > v || (ov == v && oi < i)) { v = ov; i = oi; }
-  }
+// integers in the order of the floats they come from
+__device__ __forceinline__ int rg_order(float v) { const int i = __float_as_int(v); return i ^ ((i >> 31) & 0x7fffffff); }
+// index of the warp's largest value; the lowest index wins ties
+__device__ __forceinline__ int rg_argmax(float v, int i) {
+  const int key = rg_order(v), best = __reduce_max_sync(0xffffffffu, key);
+  return static_cast<int>(__reduce_min_sync(0xffffffffu, key == best ? static_cast<unsigned>(i) : 0x7fffffffu));
 }
 
 // one warp per token; lane <-> outputs lane, lane + 32, ...
@@ -51,33 +49,34 @@ route_grouped_kernel(const float* logits, long long ld, const float* correction,
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+  const float inv = 1.f / sum;
 #pragma unroll
   for (int i = 0; i < EPL; ++i) {
     const int e = lane + 32 * i;
-    s[i] = s[i] / sum;
+    s[i] *= inv;
     c[i] = e < E ? s[i] + __ldg(correction + e) : -INFINITY;
   }
-  const int size = E / groups;
   if (keep < groups) {
+    const int size = E / groups;
+    int grp[EPL];
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) grp[i] = lane + 32 * i < E ? (lane + 32 * i) / size : -1;
     // best group first: the group of the largest remaining choice score; its members are marked and leave the race
     unsigned in = 0;                       // bit i: output lane + 32 i is in a kept group
-    float left[EPL];
-#pragma unroll
-    for (int i = 0; i < EPL; ++i) left[i] = c[i];
     for (int k = 0; k < keep; ++k) {
       float best = -INFINITY;
       int bi = 0x7fffffff;
 #pragma unroll
       for (int i = 0; i < EPL; ++i) {
         const int e = lane + 32 * i;
-        if (e < E && !(in >> i & 1u) && (left[i] > best || (left[i] == best && e < bi))) { best = left[i]; bi = e; }
+        if (e < E && !(in >> i & 1u) && (c[i] > best || (c[i] == best && e < bi))) { best = c[i]; bi = e; }
       }
-      rg_argmax(best, bi);
+      bi = rg_argmax(best, bi);
       if (bi == 0x7fffffff) break;
       const int g = bi / size;
 #pragma unroll
       for (int i = 0; i < EPL; ++i)
-        if ((lane + 32 * i) / size == g && lane + 32 * i < E) { in |= 1u << i; left[i] = -INFINITY; }
+        if (grp[i] == g) in |= 1u << i;
     }
 #pragma unroll
     for (int i = 0; i < EPL; ++i)
@@ -85,23 +84,23 @@ route_grouped_kernel(const float* logits, long long ld, const float* correction,
   }
   unsigned taken = 0;
   for (int j = 0; j < top; ++j) {
-    float best = -INFINITY, sv = 0.f;
+    float best = -INFINITY;
     int bi = 0x7fffffff;
 #pragma unroll
     for (int i = 0; i < EPL; ++i) {
       const int e = lane + 32 * i;
       if (e < E && !(taken >> i & 1u) && (c[i] > best || (c[i] == best && e < bi))) { best = c[i]; bi = e; }
     }
-    rg_argmax(best, bi);
+    bi = rg_argmax(best, bi);
+    const size_t at = static_cast<size_t>(tok) * top + j;
 #pragma unroll
     for (int i = 0; i < EPL; ++i)
-      if (lane + 32 * i == bi) { taken |= 1u << i; sv = s[i]; }
-    sv = __shfl_sync(0xffffffffu, sv, bi & 31);
-    if (lane == 0) {
-      const size_t at = static_cast<size_t>(tok) * top + j;
-      ids[at] = bi;
-      weights[at] = sv * scale;
-    }
+      if (lane + 32 * i == bi) {                 // the winner's lane
+        taken |= 1u << i;
+        ids[at] = bi;
+        weights[at] = s[i] * scale;
+      }
+    if (bi == 0x7fffffff && lane == 0) { ids[at] = E - 1; weights[at] = 0.f; }      // nothing eligible (no number among the scores)
   }
 }
 
@@ -125,8 +124,10 @@ extern "C" int b200_route_grouped(const float* logits, long long ld, const float
   if (M <= 0) return 0;
   if (!logits || !correction || !ids || !weights || E <= 0 || E > 1024 || top <= 0 || groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups)) return -1;
   const dim3 grid((M + RG_WARPS - 1) / RG_WARPS), block(32 * RG_WARPS);
+  // (3: a router of 64 experts and a few identity outputs)
   if (E <= 32) launch_ex(route_grouped_kernel<1>, grid, block, 0, stream, 0, logits, ld, correction, M, E, top, groups, keep, scale, ids, weights);
   else if (E <= 64) launch_ex(route_grouped_kernel<2>, grid, block, 0, stream, 0, logits, ld, correction, M, E, top, groups, keep, scale, ids, weights);
+  else if (E <= 96) launch_ex(route_grouped_kernel<3>, grid, block, 0, stream, 0, logits, ld, correction, M, E, top, groups, keep, scale, ids, weights);
   else if (E <= 128) launch_ex(route_grouped_kernel<4>, grid, block, 0, stream, 0, logits, ld, correction, M, E, top, groups, keep, scale, ids, weights);
   else if (E <= 256) launch_ex(route_grouped_kernel<8>, grid, block, 0, stream, 0, logits, ld, correction, M, E, top, groups, keep, scale, ids, weights);
   else launch_ex(route_grouped_kernel<32>, grid, block, 0, stream, 0, logits, ld, correction, M, E, top, groups, keep, scale, ids, weights);
