@@ -7,11 +7,13 @@
 // dimensions - the same operand tile, once K-major and once MN-major.  Tiles are 128 keys (512 + 64 columns x 128 keys are
 // 144 KB) where the queries leave room for one, else 64: the score MMA then still has 128 rows, and the upper half, whatever lies
 // behind the operand, is never read back.
-//   warp 0      TMA producer: a tile is 8 or 4 pages, in slots of 128 latent columns and one of the rotated part, each
+//   warps 0, 1  TMA producers, each for one of a slot's two 64-column chunks (a page is a box of its own and issuing one takes
+//               some 50 cycles, so one warp alone cannot feed an SM): a tile is 8 or 4 pages, in slots of 128 latent columns and one of the rotated part, each
 //               released as soon as its last product is done (rings).  In decoding the tiles of earlier tokens are requested before the dependency
 //               wait: only the new token's row is written by a kernel that may still run.
-//   warp 1      MMA issuer; where two tiles fit, the scores of the next tile go before the values of this one
-//   warps 2..9  softmax with keys on the lanes: a warp holds 32 keys of half the rows; maxima by warp reduction and through
+//   warp 2      MMA issuer; the scores of the next tile go before the values of this one as far as its slots are there (entirely
+//               where two tiles fit)
+//   warps 3..10 softmax with keys on the lanes: a warp holds 32 keys of half the rows; maxima by warp reduction and through
 //               shared memory, sums stay with their keys until the end.  They also turn the queries' second part, and keep the
 //               accumulated values (128 dimensions x N per block) in registers.
 // The splits of one row tile are a thread-block cluster that merges through distributed shared memory.  All waits are bounded.
@@ -22,7 +24,7 @@
 
 namespace b200 {
 
-constexpr int AL_THREADS = 320, AL_SOFTMAX = 256, AL_PS = 16;
+constexpr int AL_THREADS = 352, AL_SOFTMAX = 256, AL_SOFTMAX0 = 96, AL_PS = 16;
 constexpr int AL_MAX_SMEM = 232448, AL_MAX_SLOTS = 12, AL_MAX_ROT = 3;
 constexpr float AL_LOG2E = 1.4426950408889634f;
 
@@ -118,12 +120,12 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   const int ta = static_cast<int>(static_cast<long long>(n_tiles) * split / S), nt = static_cast<int>(static_cast<long long>(n_tiles) * (split + 1) / S) - ta;
 
   if (tid == 0) {
-    for (int i = 0; i < B_COUNT; ++i) mbar_init(bar(i), i == B_PFULL || i == B_QROT ? AL_SOFTMAX : 1);
+    for (int i = 0; i < B_COUNT; ++i) mbar_init(bar(i), i == B_PFULL || i == B_QROT ? AL_SOFTMAX / 32 : (i >= B_CFULL && i < B_CEMPTY) || (i >= B_RFULL && i < B_REMPTY) ? 2 : 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
   if (tid < N) sh.pos[tid] = start + min(g0 + tid, len * H - 1) / H;
-  if (warp == 1) { tmem_alloc(smem_u32(&sh.tmem), TMEM_COLS); tmem_relinquish(); }
+  if (warp == 2) { tmem_alloc(smem_u32(&sh.tmem), TMEM_COLS); tmem_relinquish(); }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -133,7 +135,7 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 #pragma unroll
   for (int i = 0; i < N; ++i) o[0][i] = o[1][i] = 0.f;
 
-  if (warp == 0) {
+  if (warp < 2) {
     const int* pt = p.c.page_table + static_cast<size_t>(seq) * p.c.max_pages;
     auto page_of = [&](int t) {                          // lane <-> page of tile t; past the last key: out of range, arrives as zeros
       const int tok = t * AL_KEYS + (lane % PAGES) * AL_PS;
@@ -145,40 +147,39 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     int cs = 0, rs = 0;
     uint32_t cp = 0, rp = 0;
     int page = nt > 0 ? page_of(ta) : 0;
+    // one chunk (if this warp has one of this slot) of the tile's pages
+    auto fetch = [&](int full, int empty_bar, uint32_t phase, uint32_t dst, const CUtensorMap* map, int chunk, int chunks) -> bool {
+      if (!__all_sync(0xffffffffu, mbar_wait(bar(empty_bar), phase ^ 1u, abort_flag, p.status, (ST_TIMEOUT_SMEM_EMPTY | (18 << 8)), limit))) return false;
+      const bool has = chunk < chunks;
+      if (lane == 0) { if (has) mbar_expect_tx(bar(full), AL_CHUNK); else mbar_arrive(bar(full)); }
+      __syncwarp();
+      if (has && lane < PAGES) tma_load_3d(dst + warp * AL_CHUNK + lane * 2048, map, bar(full), chunk * 64, 0, page);
+      return true;
+    };
     for (int j = 0; j < nt && ok; ++j) {
       if (!waited && (ta + j + 1) * AL_KEYS > last_pos) { pdl_wait(); waited = true; }      // holds the new token
       const int next = j + 1 < nt ? page_of(ta + j + 1) : 0;
-      for (int d = 0; d < nd; ++d) {
-        const int chunks = min(2, kq - 2 * d);
-        ok = __all_sync(0xffffffffu, mbar_wait(bar(B_CEMPTY + cs), cp ^ 1u, abort_flag, p.status, (ST_TIMEOUT_SMEM_EMPTY | (18 << 8)), limit));
-        if (!ok) break;
-        if (lane == 0) mbar_expect_tx(bar(B_CFULL + cs), chunks * AL_CHUNK);
-        __syncwarp();
-        // the first lanes fetch the first chunk's pages, the next ones the second's
-        if (lane < PAGES * chunks)
-          tma_load_3d(sC + cs * AL_SLOT + (lane / PAGES) * AL_CHUNK + (lane % PAGES) * 2048, &tmap_c, bar(B_CFULL + cs), (2 * d + lane / PAGES) * 64, 0, page);
-        if (++cs == p.slots) { cs = 0; cp ^= 1u; }
-      }
-      if (ok && rc > 0) {
-        ok = __all_sync(0xffffffffu, mbar_wait(bar(B_REMPTY + rs), rp ^ 1u, abort_flag, p.status, (ST_TIMEOUT_SMEM_EMPTY | (18 << 8)), limit));
-        if (!ok) break;
-        if (lane == 0) mbar_expect_tx(bar(B_RFULL + rs), rc * AL_CHUNK);
-        __syncwarp();
-        if (lane < PAGES * rc)
-          tma_load_3d(sR + rs * rc * AL_CHUNK + (lane / PAGES) * AL_CHUNK + (lane % PAGES) * 2048, &tmap_r, bar(B_RFULL + rs), (lane / PAGES) * 64, 0, page);
+      if (rc > 0) {
+        ok = fetch(B_RFULL + rs, B_REMPTY + rs, rp, sR + rs * rc * AL_CHUNK, &tmap_r, warp, rc);
         if (++rs == p.rot_slots) { rs = 0; rp ^= 1u; }
+      }
+      for (int d = 0; d < nd && ok; ++d) {
+        ok = fetch(B_CFULL + cs, B_CEMPTY + cs, cp, sC + cs * AL_SLOT, &tmap_c, 2 * d + warp, kq);
+        if (++cs == p.slots) { cs = 0; cp ^= 1u; }
       }
       page = next;
     }
     if (!ok) { const uint64_t t0 = globaltimer_ns(); while (globaltimer_ns() - t0 < 2000000ull) { } }   // copies in flight land
     if (!waited) pdl_wait();
     __syncwarp();
-  } else if (warp == 1) {
+  } else if (warp == 2) {
     pdl_wait();
-    if (lane == 0 && nt > 0) {
+    // The whole warp walks the loops, so that descriptors stay in uniform registers; one elected thread issues.
+    if (nt > 0) {
+      const bool one = elect_one();
       constexpr uint32_t IDESC_S = umma_idesc_bf16(128, N, 0, 0), IDESC_O = umma_idesc_bf16(128, N, 1, 0);      // C^T is MN-major
-      mbar_expect_tx(bar(B_Q), kq * QCHUNK);
-      for (int c = 0; c < kq; ++c) tma_load_3d(sQ + c * QCHUNK, &tmap_q, bar(B_Q), c * 64, row0 * H + g0, 0);
+      if (one) mbar_expect_tx(bar(B_Q), kq * QCHUNK);
+      for (int c = 0; c < kq; ++c) if (one) tma_load_3d(sQ + c * QCHUNK, &tmap_q, bar(B_Q), c * 64, row0 * H + g0, 0);
       const int c_steps = (rank + 15) >> 4, r_steps = (rot + 15) >> 4;
       int cs = 0, rs = 0, vs = 0;                        // slots: scores read cs, values vs
       uint32_t cp = 0, rp = 0;
@@ -186,39 +187,42 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       // (the address field counts 16 bytes).
       const uint64_t c_desc = umma_desc_k_sw128(sC), ct_desc = umma_desc_mn_sw128(sC, AL_CHUNK, 1024), r_desc = umma_desc_k_sw128(sR),
                      q_desc = umma_desc_k_sw128(sQ), qr_desc = umma_desc_k_sw128(sQ + kq * QCHUNK), p_desc = umma_desc_k_sw128(sP);
-      auto issue_s = [&](int j) -> bool {
+      // Scores of tile j: (first:) the rotated part, and slots [d0, d1).  A tile's first slots are there before the values of the tile before
+      // have freed the others, so their products go first.
+      auto issue_s = [&](int j, bool first, int d0, int d1) -> bool {
         const uint32_t d_tmem = tmem_base + (j & 1) * N;
-        for (int d = 0; d < nd; ++d) {
+        if (first && rc > 0) {
+          if (!mbar_wait(bar(B_RFULL + rs), rp, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (18 << 8)), limit)) return false;
+          tc_fence_after();
+          const uint64_t a = r_desc + static_cast<uint32_t>(rs * rc * (AL_CHUNK >> 4));
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk)
+            if (kk < r_steps && one)
+              umma_f16_ss(d_tmem, a + ((kk >> 2) * (AL_CHUNK >> 4) + 2 * (kk & 3)), qr_desc + ((kk >> 2) * (QCHUNK >> 4) + 2 * (kk & 3)), IDESC_S, kk > 0 ? 1u : 0u);
+          if (one) umma_commit(bar(B_REMPTY + rs));
+          if (++rs == p.rot_slots) { rs = 0; rp ^= 1u; }
+        }
+        for (int d = d0; d < d1; ++d) {
           if (!mbar_wait(bar(B_CFULL + cs), cp, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (18 << 8)), limit)) return false;
           tc_fence_after();
           const int steps = c_steps - 8 * d;
           const uint64_t a = c_desc + static_cast<uint32_t>(cs * (AL_SLOT >> 4)), bq = q_desc + static_cast<uint32_t>(d * (2 * QCHUNK >> 4));
 #pragma unroll
           for (int kk = 0; kk < 8; ++kk)
-            if (kk < steps)
+            if (kk < steps && one)
               umma_f16_ss(d_tmem, a + ((kk >> 2) * (AL_CHUNK >> 4) + 2 * (kk & 3)), bq + ((kk >> 2) * (QCHUNK >> 4) + 2 * (kk & 3)), IDESC_S,
-                          kk > 0 ? 1u : (d > 0 ? 1u : 0u));
+                          kk > 0 || rc > 0 || d > 0 ? 1u : 0u);
           if (++cs == p.slots) { cs = 0; cp ^= 1u; }
         }
-        if (rc > 0) {
-          if (!mbar_wait(bar(B_RFULL + rs), rp, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (18 << 8)), limit)) return false;
-          tc_fence_after();
-          const uint64_t a = r_desc + static_cast<uint32_t>(rs * rc * (AL_CHUNK >> 4));
-#pragma unroll
-          for (int kk = 0; kk < 8; ++kk)
-            if (kk < r_steps)
-              umma_f16_ss(d_tmem, a + ((kk >> 2) * (AL_CHUNK >> 4) + 2 * (kk & 3)), qr_desc + ((kk >> 2) * (QCHUNK >> 4) + 2 * (kk & 3)), IDESC_S, 1u);
-          umma_commit(bar(B_REMPTY + rs));
-          if (++rs == p.rot_slots) { rs = 0; rp ^= 1u; }
-        }
-        umma_commit(bar(B_SFULL + (j & 1)));
+        if (d1 == nd && one) umma_commit(bar(B_SFULL + (j & 1)));
         return true;
       };
+      const int early = p.ahead ? nd : min(nd - 1, p.slots - nd);
       bool ok = mbar_wait(bar(B_Q), 0, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (18 << 8)), limit) &&
                 mbar_wait(bar(B_QROT), 0, abort_flag, p.status, (ST_TIMEOUT_PEER_FLAG | (18 << 8)), limit);
-      if (ok) { tc_fence_after(); ok = issue_s(0); }
+      if (ok) { tc_fence_after(); ok = issue_s(0, true, 0, nd); }
       for (int j = 0; j < nt && ok; ++j) {
-        if (p.ahead && j + 1 < nt && !issue_s(j + 1)) { ok = false; break; }
+        if (j + 1 < nt && !issue_s(j + 1, true, 0, early)) { ok = false; break; }
         if (!mbar_wait(bar(B_PFULL), j & 1u, abort_flag, p.status, (ST_TIMEOUT_PEER_FLAG | (18 << 8)), limit)) { ok = false; break; }
         tc_fence_after();
         const uint64_t bp = p_desc + (p.ahead ? static_cast<uint32_t>((j & 1) * (PCHUNKS * QCHUNK >> 4)) : 0u);
@@ -227,19 +231,19 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
           const uint64_t a = ct_desc + static_cast<uint32_t>(vs * (AL_SLOT >> 4));
 #pragma unroll
           for (int kk = 0; kk < KEYS / 16; ++kk)
-            umma_f16_ss(d_tmem, a + kk * (2048 >> 4), bp + ((kk >> 2) * (QCHUNK >> 4) + 2 * (kk & 3)), IDESC_O, kk > 0 ? 1u : 0u);
-          umma_commit(bar(B_CEMPTY + vs));
+            if (one) umma_f16_ss(d_tmem, a + kk * (2048 >> 4), bp + ((kk >> 2) * (QCHUNK >> 4) + 2 * (kk & 3)), IDESC_O, kk > 0 ? 1u : 0u);
+          if (one) umma_commit(bar(B_CEMPTY + vs));
           if (++vs == p.slots) vs = 0;
         }
-        umma_commit(bar(B_OFULL + (j & 1)));
-        if (!p.ahead && j + 1 < nt && !issue_s(j + 1)) { ok = false; break; }
+        if (one) umma_commit(bar(B_OFULL + (j & 1)));
+        if (early < nd && j + 1 < nt && !issue_s(j + 1, false, early, nd)) { ok = false; break; }
       }
     }
     __syncwarp();
   } else {
     pdl_wait();
-    const int qd = warp & 3, half = (warp - 2) >> 2, c0 = half * NC;      // key quarter = TMEM lane quarter; first column
-    const int st = tid - 64;
+    const int qd = warp & 3, half = (warp - 3) >> 2, c0 = half * NC;      // key quarter = TMEM lane quarter; first column
+    const int st = tid - AL_SOFTMAX0;
     // the queries' rotated part; columns up to the end of its chunks and rows beyond the portion are zero
     const int np = p.d.true_rot / 2, wide = rc * 32;
     for (int i = st; i < N * wide; i += AL_SOFTMAX) {
@@ -255,7 +259,8 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       *reinterpret_cast<__nv_bfloat162*>(pQr + (j >> 5) * QCHUNK + al_swizzled(r, (2 * j) & 63)) = __floats2bfloat162_rn(u, v);
     }
     fence_proxy_async_smem();
-    mbar_arrive(bar(B_QROT));
+    __syncwarp();
+    if (lane == 0) mbar_arrive(bar(B_QROT));
 
     const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(qd * 32) << 16);
     float m_run[NC], l_run[NC];
@@ -346,7 +351,8 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       if (qd == 0 && lane < NC) sh.alpha[turn][c0 + lane] = a_mine;
       tc_fence_before();
       fence_proxy_async_smem();
-      mbar_arrive(bar(B_PFULL));
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar(B_PFULL));          // one arrival per warp: they queue up at the barrier
       if (j > 0 && !o_update(j - 1)) ok = false;
     }
     named_bar_sync(1, AL_SOFTMAX);                       // the last turn's factors are written
@@ -365,8 +371,8 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   __syncthreads();                                       // all products are done: the rings become the merge buffer
   float* obuf = reinterpret_cast<float*>(al_smem);
   const int OP = rank + 4;
-  if (warp >= 2) {
-    const int half = (warp - 2) >> 2, at = (warp & 3) * 32 + lane;
+  if (warp >= 3) {
+    const int half = (warp - 3) >> 2, at = (warp & 3) * 32 + lane;
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
       const int dim = (half + 2 * k) * 128 + at;
@@ -375,8 +381,9 @@ attn_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         for (int i = 0; i < N; ++i) obuf[i * OP + dim] = o[k][i];
       }
     }
-    if (tid - 64 < N) sh.l[tid - 64] = sh.lw[0][tid - 64] + sh.lw[1][tid - 64] + sh.lw[2][tid - 64] + sh.lw[3][tid - 64];
-  } else if (warp == 1) {
+    const int c = tid - AL_SOFTMAX0;
+    if (c < N) sh.l[c] = sh.lw[0][c] + sh.lw[1][c] + sh.lw[2][c] + sh.lw[3][c];
+  } else if (warp == 2) {
     tc_fence_after();
     tmem_dealloc(tmem_base, TMEM_COLS);
   }
@@ -433,9 +440,9 @@ static bool al_plan(int rank, int rot, int n, AlPlan& plan) {
       auto bytes = [&](int slots, int rs) { return slots * keys * 256 + rs * rc * keys * 128 + (kq + rc) * n * 128 + (ahead ? 2 : 1) * (keys / 64) * n * 128 + tail; };
       int slots = ahead ? 2 * nd : nd, rs = 1;
       if (bytes(slots, rs) > AL_MAX_SMEM) continue;
-      // a third tile of the rotated part only beside a third tile of latents
+      // a spare slot first, then a second tile of the rotated part; a third one only beside a third tile of latents
       while (true) {
-        if (rs < 2 && bytes(slots, rs + 1) <= AL_MAX_SMEM) ++rs;
+        if (rs < 2 && slots > nd && bytes(slots, rs + 1) <= AL_MAX_SMEM) ++rs;
         else if (slots < AL_MAX_SLOTS && bytes(slots + 1, rs) <= AL_MAX_SMEM) ++slots;
         else if (rs < AL_MAX_ROT && slots >= 3 * nd && bytes(slots, rs + 1) <= AL_MAX_SMEM) ++rs;
         else break;

@@ -70,7 +70,7 @@ attn_prefill_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
   const uint64_t limit = p.limit_ns;
 
   if (threadIdx.x == 0) {
-    for (int i = 0; i < B_COUNT; ++i) mbar_init(bar(i), i == B_PFULL ? PL_SOFTMAX : 1);
+    for (int i = 0; i < B_COUNT; ++i) mbar_init(bar(i), i == B_PFULL ? PL_SOFTMAX / 32 : 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
@@ -108,13 +108,15 @@ attn_prefill_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
     }
     __syncwarp();
   } else if (warp == 1) {
-    if (lane == 0) {
+    // The whole warp walks the loops, so that descriptors stay in uniform registers; one elected thread issues.
+    {
+      const bool one = elect_one();
       constexpr uint32_t IDESC_S = umma_idesc_bf16(128, 128, 0, 0);
       const uint32_t idesc_pv = umma_idesc_bf16(128, dv16, 0, 1);        // B (= V) is MN-major
       const int n_steps = (p.dn + 15) >> 4, r_steps = (p.dr + 15) >> 4;
       int ks = 0, vs = 0;
       uint32_t kp = 0, vp = 0;
-      // one thread issues everything: a descriptor costs an addition (the address field counts 16 bytes)
+      // a descriptor costs an addition (the address field counts 16 bytes)
       const uint64_t q_desc = umma_desc_k_sw128(sQ), k_desc = umma_desc_k_sw128(sK), p_desc = umma_desc_k_sw128(sP), v_desc = umma_desc_mn_sw128(sV, PL_CHUNK, 1024);
       auto issue_s = [&](int j) {                                        // the K stage has been waited for
         const uint32_t d = tmem_base + (j & 1) * 128;
@@ -124,10 +126,9 @@ attn_prefill_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
           const uint32_t off = c * (PL_CHUNK >> 4);
 #pragma unroll
           for (int kk = 0; kk < 4; ++kk)
-            if (kk < steps) umma_f16_ss(d, q_desc + (off + 2 * kk), kd + (off + 2 * kk), IDESC_S, kk > 0 ? 1u : (c > 0 ? 1u : 0u));
+            if (kk < steps && one) umma_f16_ss(d, q_desc + (off + 2 * kk), kd + (off + 2 * kk), IDESC_S, kk > 0 ? 1u : (c > 0 ? 1u : 0u));
         }
-        umma_commit(bar(B_KEMPTY + ks));
-        umma_commit(bar(B_SFULL + (j & 1)));
+        if (one) { umma_commit(bar(B_KEMPTY + ks)); umma_commit(bar(B_SFULL + (j & 1))); }
         if (++ks == p.k_stages) { ks = 0; kp ^= 1u; }
       };
       bool ok = mbar_wait(bar(B_QFULL), 0, abort_flag, p.status, (ST_TIMEOUT_SMEM_FULL | (19 << 8)), limit) &&
@@ -146,9 +147,8 @@ attn_prefill_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
         const uint64_t a = p_desc + (p.p_stages == 2 ? static_cast<uint32_t>((j & 1) * (2 * PL_CHUNK >> 4)) : 0u), bv = v_desc + static_cast<uint32_t>(vs * (v_bytes >> 4));
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk)
-          umma_f16_ss(d, a + ((kk >> 2) * (PL_CHUNK >> 4) + 2 * (kk & 3)), bv + kk * (2048 >> 4), idesc_pv, kk > 0 ? 1u : 0u);
-        umma_commit(bar(B_VEMPTY + vs));
-        umma_commit(bar(B_OFULL + (j & 1)));
+          if (one) umma_f16_ss(d, a + ((kk >> 2) * (PL_CHUNK >> 4) + 2 * (kk & 3)), bv + kk * (2048 >> 4), idesc_pv, kk > 0 ? 1u : 0u);
+        if (one) { umma_commit(bar(B_VEMPTY + vs)); umma_commit(bar(B_OFULL + (j & 1))); }
         if (++vs == p.v_stages) { vs = 0; vp ^= 1u; }
       }
     }
@@ -239,7 +239,8 @@ attn_prefill_latent_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       m_run = m_new;
       tc_fence_before();
       fence_proxy_async_smem();
-      mbar_arrive(bar(B_PFULL));
+      __syncwarp();
+      if (lane == 0) mbar_arrive(bar(B_PFULL));         // one arrival per warp: they queue up at the barrier
       if (j > 0 && !o_update(j - 1, alpha_prev)) { ok = false; continue; }
       alpha_prev = alpha;
     }
