@@ -216,39 +216,44 @@ def kernels(z: dict, batch=32, ctx=1024, seqs=4, prompt=2048) -> dict:
         del zxg, stream, h
         torch.cuda.empty_cache()
 
-    # attention: decoding over the paged cache
+    # attention: decoding over the paged cache, a short and a long context
     G = max(1, H // 4)
-    mp = ctx // 16
-    table = torch.arange(batch * mp, dtype=torch.int32, device="cuda").view(batch, mp)
-    pos = torch.full((batch,), ctx - 1, dtype=torch.int32, device="cuda")
-    lens = pos + 1
     dm = LT.dims(H, rank, r)
-    caches = [A.PagedKVCache(batch * mp, 1, 16, "cuda", dk=rank + r, dv=0) for _ in range(8)]
-    for c in caches:
-        c.data.normal_()
-    cos, sin = A.rope_tables(max(ctx, prompt), 1e6, "cuda", r)
-    qa, q = rnd(batch, H * rank), rnd(batch, H * (n + r))
-    scale = (n + r) ** -0.5
-    put("decode", "rakelorn attention", per_launch(lambda l: LT.attend(qa, q[:, n:], n + r, dm, scale, pos, None, cos, sin, caches[l], table, seq_lens=lens), 8),
-        batch * ctx * (rank + r) * 2 + batch * H * (2 * rank + r) * 2, 2.0 * batch * ctx * H * (2 * rank + r))
-    low = rnd(batch, qr + rank + r + H, dtype=torch.float32)
-    gq, gc = torch.ones(qr, device="cuda"), torch.ones(rank, device="cuda")
-    put("decode", "rakelorn norms + cache append", per_launch(lambda l: LT.append(low, qr, gq, gc, 1e-6, dm, pos, None, cos, sin, caches[l], table, seq_lens=lens), 8),
-        batch * (qr + rank + r) * 6)
-    del caches
-    caches = [A.PagedKVCache(batch * mp, G, 16, "cuda") for _ in range(8)]
-    for c in caches:
-        c.data.normal_()
     qkv_n = (H + 2 * G) * 128
-    qkvg = rnd(batch, D.padded(qkv_n + H))
     sink = torch.zeros(H, device="cuda")
-    c2, s2 = A.rope_tables(max(ctx, prompt), 1e4, "cuda", 64)
-    out = torch.empty((batch, H * 128), dtype=bf, device="cuda")
-    spec = A.attn_spec(128 ** -0.5, chunk=8192, sink=sink, gate=qkvg[:, qkv_n:qkv_n + H])
-    put("decode", "volonex attention (rotary, append, sink, gate)", per_launch(lambda l: A.attn_decode_paged(qkvg, H, pos, lens, c2, s2, caches[l], table, spec, out), 8),
-        batch * ctx * G * 512, 4.0 * batch * ctx * H * 128)
-    del caches
-    torch.cuda.empty_cache()
+    scale = (n + r) ** -0.5
+    gq, gc = torch.ones(qr, device="cuda"), torch.ones(rank, device="cuda")
+    for c_len, reps in ((ctx, 8), (8 * ctx, 2)):
+        note_ctx = f", {c_len} keys"
+        mp = c_len // 16
+        table = torch.arange(batch * mp, dtype=torch.int32, device="cuda").view(batch, mp)
+        pos = torch.full((batch,), c_len - 1, dtype=torch.int32, device="cuda")
+        lens = pos + 1
+        caches = [A.PagedKVCache(batch * mp, 1, 16, "cuda", dk=rank + r, dv=0) for _ in range(reps)]
+        for c in caches:
+            c.data.normal_()
+        cos, sin = A.rope_tables(c_len, 1e6, "cuda", r)
+        qa, q = rnd(batch, H * rank), rnd(batch, H * (n + r))
+        put("decode", "rakelorn attention" + note_ctx, per_launch(lambda l: LT.attend(qa, q[:, n:], n + r, dm, scale, pos, None, cos, sin, caches[l % reps], table, seq_lens=lens), 8),
+            batch * c_len * (rank + r) * 2 + batch * H * (2 * rank + r) * 2, 2.0 * batch * c_len * H * (2 * rank + r))
+        if c_len == ctx:
+            low = rnd(batch, qr + rank + r + H, dtype=torch.float32)
+            put("decode", "rakelorn norms + cache append", per_launch(lambda l: LT.append(low, qr, gq, gc, 1e-6, dm, pos, None, cos, sin, caches[l], table, seq_lens=lens), 8),
+                batch * (qr + rank + r) * 6)
+        del caches
+        caches = [A.PagedKVCache(batch * mp, G, 16, "cuda") for _ in range(reps)]
+        for c in caches:
+            c.data.normal_()
+        qkvg = rnd(batch, D.padded(qkv_n + H))
+        c2, s2 = A.rope_tables(c_len, 1e4, "cuda", 64)
+        out = torch.empty((batch, H * 128), dtype=bf, device="cuda")
+        spec = A.attn_spec(128 ** -0.5, sink=sink, gate=qkvg[:, qkv_n:qkv_n + H])
+        put("decode", "volonex attention (rotary, append, sink, gate)" + note_ctx, per_launch(lambda l: A.attn_decode_paged(qkvg, H, pos, lens, c2, s2, caches[l % reps], table, spec, out), 8),
+            batch * c_len * G * 512, 4.0 * batch * c_len * H * 128)
+        del caches
+        torch.cuda.empty_cache()
+    c2, s2 = A.rope_tables(prompt, 1e4, "cuda", 64)
+    cos, sin = A.rope_tables(prompt, 1e6, "cuda", r)
     # prefill, and a short portion at the end of a long context
     mp = prompt // 16
     table = torch.arange(seqs * mp, dtype=torch.int32, device="cuda").view(seqs, mp)

@@ -7,14 +7,13 @@
 #include "ptx.cuh"
 #include "api.h"
 #include "launch.cuh"
+#include "dense_epilogue.cuh"
 
 namespace b200 {
 
 template <typename T> __device__ __forceinline__ float la_f(T v);
 template <> __device__ __forceinline__ float la_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ float la_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-
-constexpr int LA_THREADS = 256;
 
 struct LatentAppendParams {
   const float* in; long long ld;
@@ -31,9 +30,9 @@ struct LatentAppendParams {
   int* status;
 };
 
-// one CTA per token
-template <typename T>
-__global__ void __launch_bounds__(LA_THREADS) latent_append_kernel(const __grid_constant__ LatentAppendParams p) {
+// one CTA per token, four columns at a time
+template <typename T, int THREADS>
+__global__ void __launch_bounds__(THREADS) latent_append_kernel(const __grid_constant__ LatentAppendParams p) {
   pdl_launch_dependents();
   pdl_wait();
   const int tok = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -42,48 +41,58 @@ __global__ void __launch_bounds__(LA_THREADS) latent_append_kernel(const __grid_
   // a position outside the tables or the sequence's pages must not become a stray write: skipped and reported
   bool bad = pos < 0 || pos >= p.max_pos || seq < 0 || seq >= p.c.num_seqs || pos / ps >= p.c.max_pages;
   int page = 0;
-  if (!bad && !empty) {
-    page = p.c.page_table[static_cast<size_t>(seq) * p.c.max_pages + pos / ps];
-    bad = page < 0 || page >= p.c.num_pages;
-  }
-  if (bad && threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, static_cast<int>(ST_BAD_ARGUMENT) | (15 << 8));
+  if (!bad && !empty) page = p.c.page_table[static_cast<size_t>(seq) * p.c.max_pages + pos / ps];
   const float* row = p.in + static_cast<size_t>(tok) * p.ld;
   const float* lat_in = row + p.q_rank;
   const float* rot_in = lat_in + p.d.rank;
+  auto squares = [](float4 v, int left) {               // of the first `left` of four
+    return (left > 0 ? v.x * v.x : 0.f) + (left > 1 ? v.y * v.y : 0.f) + (left > 2 ? v.z * v.z : 0.f) + (left > 3 ? v.w * v.w : 0.f);
+  };
   float sq = 0.f, sc = 0.f;
-  for (int i = threadIdx.x; i < p.true_q_rank; i += LA_THREADS) sq += row[i] * row[i];
-  for (int i = threadIdx.x; i < p.d.true_rank; i += LA_THREADS) sc += lat_in[i] * lat_in[i];
+#pragma unroll 4
+  for (int i = threadIdx.x * 4; i < p.q_rank; i += THREADS * 4) sq += squares(*reinterpret_cast<const float4*>(row + i), p.true_q_rank - i);
+#pragma unroll 2
+  for (int i = threadIdx.x * 4; i < p.d.rank; i += THREADS * 4) sc += squares(*reinterpret_cast<const float4*>(lat_in + i), p.d.true_rank - i);
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) { sq += __shfl_xor_sync(0xffffffffu, sq, o); sc += __shfl_xor_sync(0xffffffffu, sc, o); }
-  __shared__ float red[2][LA_THREADS / 32];
+  __shared__ float red[2][THREADS / 32];
   if (lane == 0) { red[0][warp] = sq; red[1][warp] = sc; }
   __syncthreads();
   sq = sc = 0.f;
 #pragma unroll
-  for (int w = 0; w < LA_THREADS / 32; ++w) { sq += red[0][w]; sc += red[1][w]; }
+  for (int w = 0; w < THREADS / 32; ++w) { sq += red[0][w]; sc += red[1][w]; }
   const float fq = 1.f / sqrtf(sq / static_cast<float>(p.true_q_rank) + p.eps), fc = 1.f / sqrtf(sc / static_cast<float>(p.d.true_rank) + p.eps);
-  T* cq = static_cast<T*>(p.cq) + static_cast<size_t>(tok) * p.ldq;
-  for (int i = threadIdx.x; i < p.q_rank; i += LA_THREADS) cq[i] = static_cast<T>(i < p.true_q_rank ? row[i] * fq * __ldg(p.q_gain + i) : 0.f);
+  bad = bad || (!empty && (page < 0 || page >= p.c.num_pages));
+  if (bad && threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, static_cast<int>(ST_BAD_ARGUMENT) | (15 << 8));
 
-  const int dk = p.d.rank + p.d.rot;
-  T* rec = bad || empty ? nullptr : static_cast<T*>(p.c.data) + (static_cast<size_t>(page) * ps + pos % ps) * dk;
-  T* lat = p.lat ? static_cast<T*>(p.lat) + static_cast<size_t>(tok) * dk : nullptr;
-  auto put = [&](int i, float v) {
-    const T t = static_cast<T>(v);
-    if (rec) rec[i] = t;
-    if (lat) lat[i] = t;
+  constexpr bool F32 = sizeof(T) == 4;
+  auto scaled = [](float4 v, float f, float4 g) { return make_float4(v.x * f * g.x, v.y * f * g.y, v.z * f * g.z, v.w * f * g.w); };
+  auto cut = [](float4 v, int left) {                   // padding is zero whatever the linear left there
+    return make_float4(left > 0 ? v.x : 0.f, left > 1 ? v.y : 0.f, left > 2 ? v.z : 0.f, left > 3 ? v.w : 0.f);
   };
-  for (int i = threadIdx.x; i < p.d.rank; i += LA_THREADS) put(i, i < p.d.true_rank ? lat_in[i] * fc * __ldg(p.c_gain + i) : 0.f);
+#pragma unroll 4
+  for (int i = threadIdx.x * 4; i < p.q_rank; i += THREADS * 4)
+    store4_any(p.cq, F32, static_cast<long long>(tok) * p.ldq + i,
+               scaled(cut(*reinterpret_cast<const float4*>(row + i), p.true_q_rank - i), fq, __ldg(reinterpret_cast<const float4*>(p.q_gain + i))));
+  const int dk = p.d.rank + p.d.rot;
+  const long long rec = (static_cast<long long>(page) * ps + pos % ps) * dk;
+  const bool keep = !bad && !empty;
+  auto put = [&](int i, float4 v) {
+    if (keep) store4_any(p.c.data, F32, rec + i, v);
+    if (p.lat) store4_any(p.lat, F32, static_cast<long long>(tok) * dk + i, v);
+  };
+#pragma unroll 2
+  for (int i = threadIdx.x * 4; i < p.d.rank; i += THREADS * 4)
+    put(i, scaled(cut(*reinterpret_cast<const float4*>(lat_in + i), p.d.true_rank - i), fc, __ldg(reinterpret_cast<const float4*>(p.c_gain + i))));
+  // the last threads take the rotated part: they had the least to do
   const int np = p.d.true_rot / 2, at = bad ? 0 : pos;
-  for (int j = threadIdx.x; j < p.d.rot / 2; j += LA_THREADS) {
-    float u = 0.f, v = 0.f;
-    if (j < np) {
-      const float c = p.cos_tab[static_cast<size_t>(at) * np + j], s = p.sin_tab[static_cast<size_t>(at) * np + j];
-      u = rot_in[2 * j] * c - rot_in[2 * j + 1] * s;
-      v = rot_in[2 * j + 1] * c + rot_in[2 * j] * s;
-    }
-    put(p.d.rank + 2 * j, u);
-    put(p.d.rank + 2 * j + 1, v);
+  for (int i = (THREADS - 1 - threadIdx.x) * 4; i < p.d.rot; i += THREADS * 4) {
+    const float4 x = *reinterpret_cast<const float4*>(rot_in + i);
+    const size_t t = static_cast<size_t>(at) * np + i / 2;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i / 2 < np) { const float c = p.cos_tab[t], s = p.sin_tab[t]; o.x = x.x * c - x.y * s; o.y = x.y * c + x.x * s; }
+    if (i / 2 + 1 < np) { const float c = p.cos_tab[t + 1], s = p.sin_tab[t + 1]; o.z = x.z * c - x.w * s; o.w = x.w * c + x.z * s; }
+    put(p.d.rank + i, o);
   }
 }
 
@@ -145,13 +154,17 @@ extern "C" int b200_latent_append(const float* in, long long ld, int M, int q_ra
   if (M <= 0) return 0;
   if (!latent_cache_ok(cache, dims)) return -1;
   if (!in || !cq || !q_gain || !c_gain || !positions || q_rank <= 0 || true_q_rank <= 0 || true_q_rank > q_rank || ldq < q_rank) return -2;
+  auto al16 = [](const void* a) { return (reinterpret_cast<uintptr_t>(a) & 15) == 0; };
+  if (q_rank % 8 || ld % 4 || ldq % 8 || !al16(in) || !al16(cq) || !al16(q_gain) || !al16(c_gain) || !al16(lat)) return -4;
   if (ld < q_rank + cache->dk || max_pos <= 0 || (dims->true_rot > 0 && (!cos_tab || !sin_tab))) return -3;
   LatentAppendParams p;
   p.in = in; p.ld = ld; p.q_rank = q_rank; p.true_q_rank = true_q_rank; p.q_gain = q_gain; p.c_gain = c_gain; p.eps = eps; p.d = *dims;
   p.positions = positions; p.seq_ids = seq_ids; p.seq_lens = seq_lens; p.cos_tab = cos_tab; p.sin_tab = sin_tab; p.max_pos = max_pos;
   p.c = *cache; p.cq = cq; p.ldq = ldq; p.lat = lat; p.status = status;
-  if (cache->f32) launch_ex(latent_append_kernel<float>, dim3(M), dim3(LA_THREADS), 0, stream, 0, p);
-  else launch_ex(latent_append_kernel<__nv_bfloat16>, dim3(M), dim3(LA_THREADS), 0, stream, 0, p);
+  // few tokens: as much of a row at once as possible
+  if (cache->f32) launch_ex(latent_append_kernel<float, 128>, dim3(M), dim3(128), 0, stream, 0, p);
+  else if (M <= 256) launch_ex(latent_append_kernel<__nv_bfloat16, 256>, dim3(M), dim3(256), 0, stream, 0, p);
+  else launch_ex(latent_append_kernel<__nv_bfloat16, 128>, dim3(M), dim3(128), 0, stream, 0, p);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -2000 - static_cast<int>(e);
 }

@@ -111,7 +111,7 @@ class LatentAttention:
             return LT.attend_expanded(q, m.heads, m.dn, m.dr, m.dv, D.linear(lat, W["ukv"]), lat[:, m.rank:], m.scale, c.cu_seqlens, ctx,
                                       c.positions, c.max_len, gate)
         qa = D.linear_heads(q, W["uk"], m.dn + m.dr, m.rank)
-        if self.in_latent_space:
+        if self.in_latent_space and (c.decode or c.max_len * m.heads <= LT.MAX_ROWS):
             keys = None if c.decode else (c.max_len if c.portions is None else max(a + n for a, n in c.portions))
             o = LT.attend(qa, q[:, m.dn:], m.dn + m.dr, self.dims, m.scale, c.positions, seq_ids, self.cos, self.sin, cache, kv.page_table,
                           cu=c.cu_seqlens, max_len=c.max_len, seq_lens=seq_lens, keys=keys)

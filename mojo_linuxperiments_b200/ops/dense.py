@@ -14,6 +14,7 @@ from . import _lib
 from .workspace import default_workspace
 
 DECODE_MAX_M = 64              # up to this many tokens the weight-streaming kernel runs
+HEADS_MAX_M = 8192             # tokens per launch of a linear per head
 
 
 def padded(n: int) -> int:
@@ -134,10 +135,15 @@ def linear_heads(x: torch.Tensor, w: GroupedW, x_group: int, y_group: int, gate:
                  out_dtype: torch.dtype | None = None, splits: int = 0) -> torch.Tensor:
     """One linear per head in one launch: group g takes columns g * x_group .. of x and writes columns g * y_group .. of the
     result; ``gate`` fp32 [M, groups] (row stride free): logits of a sigmoid on each head's result."""
+    y = rows(x.shape[0], w.groups * y_group, out_dtype or x.dtype, x.device)
+    for a in range(0, x.shape[0], HEADS_MAX_M):             # what one launch's grid can count
+        _linear_heads(x[a:a + HEADS_MAX_M], w, x_group, y_group, gate[a:a + HEADS_MAX_M] if gate is not None else None,
+                      y[a:a + HEADS_MAX_M], splits)
+    return y
+
+
+def _linear_heads(x, w, x_group, y_group, gate, y, splits) -> None:
     M = x.shape[0]
-    y = rows(M, w.groups * y_group, out_dtype or x.dtype, x.device)
-    if M == 0:
-        return y
     assert x.dtype == w.data.dtype and x.stride(1) == 1 and x_group % 8 == 0 and y_group % 8 == 0 and y_group >= (w.n + 3) // 4 * 4
     assert x.shape[1] >= (w.groups - 1) * x_group + w.k and (gate is None or gate.dtype == torch.float32)
     epi = _lib.DenseEpilogue(mode=EPI_STORE, out_f32=int(y.dtype == torch.float32), exact=int(x.dtype == torch.float32), y=y.data_ptr(),
@@ -152,7 +158,6 @@ def linear_heads(x: torch.Tensor, w: GroupedW, x_group: int, y_group: int, gate:
             x.data_ptr(), x.stride(0), w.data.data_ptr(), w.data.stride(0), M, M, w.n, w.k, ctypes.byref(epi), ctypes.byref(g),
             default_workspace(x.device).status.data_ptr(), _lib.num_sms(x.device.index), splits, _lib.stream())
         _lib.check(rc, "bf16_gemm_decode_grouped")
-    return y
 
 
 def linear_experts(x: torch.Tensor, w: GroupedW, work, act: str | None = None, force: int = 0) -> torch.Tensor:

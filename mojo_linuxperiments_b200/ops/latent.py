@@ -11,6 +11,9 @@ from .dense import rows
 from .workspace import default_workspace
 
 
+MAX_ROWS = 32 * 65535          # (token, head) pairs of a portion that ``attend`` takes
+
+
 def dims(heads: int, rank: int, rot: int) -> "_lib.LatentDims":
     up = lambda n: (n + 7) // 8 * 8
     return _lib.LatentDims(heads, up(rank), up(rot), rank, rot)

@@ -271,7 +271,7 @@ class Latents:
         self.lens, self.H, self.n, self.r, self.dv, self.q_rank, self.rank, self.dtype = lens, H, n, r, dv, q_rank, rank, DT[dtype]
         self.dn, self.dr, self.vp, self.qp, self.rp = p8(n), p8(r), p8(dv), p8(q_rank), p8(rank)
         g = gen(seed)
-        self.low = [torch.randn((t, self.qp + self.rp + self.dr + H), generator=g, device=DEV) for t in lens]
+        self.low = [torch.randn((t, p8(self.qp + self.rp + self.dr + H)), generator=g, device=DEV) for t in lens]
         self.q = [(torch.randn((t, H, self.dn + self.dr), generator=g, device=DEV)).to(self.dtype) for t in lens]
         for q in self.q:
             q[:, :, n:self.dn] = 0
@@ -311,7 +311,11 @@ class Latents:
         return cq, c, kr, q[:, :, :self.n], R.rotate_pairs(q[:, :, self.dn:self.dn + self.r], pos, self.base, self.r)
 
     def gates(self, b):
-        return self.low[b][:, self.qp + self.rp + self.dr:].double()
+        return self.gate(self.low[b]).double()
+
+    def gate(self, low):
+        at = self.qp + self.rp + self.dr
+        return low[:, at:at + self.H]
 
     def want(self, b):
         _, c, kr, qn, qr = self.parts(b)
@@ -335,7 +339,7 @@ class Latents:
         cu = i32(torch.tensor([0] + [k for _, k in spans.values()]).cumsum(0))
         longest = max(k for _, k in spans.values())
         LT.append(low, self.q_rank, self.qg, self.cg, self.eps, self.dims, pos, sid, self.cos, self.sin, self.cache, self.table)
-        gate = low[:, self.qp + self.rp + self.dr:]
+        gate = self.gate(low)
         ld = self.dn + self.dr
         if how == "expanded":
             ends = [a + k for a, k in spans.values()]
@@ -366,7 +370,7 @@ class Latents:
         else:
             LT.rotary_heads(q, self.H, self.dn + self.dr, self.dn, self.r, pos, self.cos, self.sin)
             o = LT.attend_any(qa, q[:, self.dn:], self.dn + self.dr, self.dims, self.scale, pos, None, self.cache, self.table, seq_lens=lens)
-        return self.head_values(D.linear_heads(o, self.w_uv, self.rp, self.vp, gate=low[:, self.qp + self.rp + self.dr:]))
+        return self.head_values(D.linear_heads(o, self.w_uv, self.rp, self.vp, gate=self.gate(low)))
 
 
 ATOL = {"float32": 2e-5, "bfloat16": 4e-2}
@@ -555,7 +559,13 @@ def wide() -> LC.LayeredConfig:
     return LC.LayeredConfig("Rakelorn", 331, 160, layers, 1.0, 1.0, 1e-5, LC.Loop(0, 2, 2))
 
 
-MAKES = [uneven, bare, wide, LC.tiny_rakelorn]
+def recurrent_only() -> LC.LayeredConfig:
+    """Nothing in the paged cache; a loop of one pass."""
+    layers = (LC.LayerSpec(LC.MinGRUSpec(72), LC.MoE(4, 2, 56, 1.1, 1, 5, 3)), LC.LayerSpec(LC.MinGRUSpec(130), LC.MoE(3, 2, 64, 0.6)))
+    return LC.LayeredConfig("Rakelorn", 97, 84, layers, 1.2, 1.0, 1e-6, LC.Loop(1, 2, 1))
+
+
+MAKES = [uneven, bare, wide, recurrent_only, LC.tiny_rakelorn]
 
 
 class Model:
