@@ -49,8 +49,7 @@ class KVState:
         layout = cfg.cache_layout(rt)
         size = max((_DTYPES[s.dtype].itemsize for s in layout if s is not None), default=0)
         states = sum(n for run in _states(cfg) for n in run.values()) * num_seqs * 4
-        return (sum(_record(s, rt.page_size) for s in layout) * pages * size + states + num_seqs * max_pages * 4 + num_seqs * 8 +
-                5 * 1024 + 512 * len(layout))
+        return sum(_record(s, rt.page_size) for s in layout) * pages * size + states + num_seqs * max_pages * 4 + num_seqs * 8 + 3 * 1024
 
     def __init__(self, cfg: ModelConfig, rt: RuntimeConfig, device, num_seqs: int, max_seq_len: int, alloc=None):
         """``alloc(shape, dtype) -> zeroed tensor``: where the cache lives (the rank's HBM arena); default torch.zeros.
