@@ -82,41 +82,69 @@ __global__ void __launch_bounds__(1024) moe_align_kernel(const int* ids, int M, 
 
   extern __shared__ int sm[];
   int* cnt = sm;                  // [n_local]
-  int* off = sm + n_local;        // [n_local + 1]
-  int* cur = off + n_local + 1;   // [n_local]
-  const int pairs = M * k;
-  for (int i = threadIdx.x; i < n_local; i += blockDim.x) { cnt[i] = 0; cur[i] = 0; }
+  int* cur = sm + n_local;        // [n_local] next free slot
+  __shared__ int warp_rows[32], warp_tiles[32];
+  const int pairs = M * k, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  for (int i = tid; i < n_local; i += blockDim.x) cnt[i] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    const int e = ids[i] - e0;
-    if (e >= 0 && e < n_local) atomicAdd(&cnt[e], 1);
+  // four consecutive pairs per thread and round: their loads and their atomics do not wait for one another
+  for (int i = tid * 4; i < pairs; i += blockDim.x * 4) {
+    int e[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) e[j] = i + j < pairs ? ids[i + j] - e0 : -1;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) if (e[j] >= 0 && e[j] < n_local) atomicAdd(&cnt[e[j]], 1);
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int run = 0, nt = 0;
-    for (int e = 0; e < n_local; ++e) {
-      off[e] = run;
-      for (int r = 0; r < cnt[e]; r += 128) { tiles[nt] = make_int4(e, run + r, min(128, cnt[e] - r), 0); ++nt; }
-      run += cnt[e];
+  // running sums over the experts, thread <-> expert
+  const int mine = tid < n_local ? cnt[tid] : 0, my_tiles = (mine + 127) >> 7;
+  int rows = mine, nt = my_tiles;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int r = __shfl_up_sync(0xffffffffu, rows, o), t = __shfl_up_sync(0xffffffffu, nt, o);
+    if (lane >= o) { rows += r; nt += t; }
+  }
+  if (lane == 31) { warp_rows[warp] = rows; warp_tiles[warp] = nt; }
+  __syncthreads();
+  if (warp == 0) {
+    int r = warp_rows[lane], t = warp_tiles[lane];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int ro = __shfl_up_sync(0xffffffffu, r, o), to = __shfl_up_sync(0xffffffffu, t, o);
+      if (lane >= o) { r += ro; t += to; }
     }
-    off[n_local] = run;
-    meta[0] = run;
+    warp_rows[lane] = r;
+    warp_tiles[lane] = t;
+  }
+  __syncthreads();
+  if (warp > 0) { rows += warp_rows[warp - 1]; nt += warp_tiles[warp - 1]; }
+  const int first = rows - mine;
+  if (tid < n_local) {
+    counts[tid] = mine;
+    offsets[tid] = first;
+    cur[tid] = first;
+    for (int j = 0; j < my_tiles; ++j) tiles[nt - my_tiles + j] = make_int4(tid, first + j * 128, min(128, mine - j * 128), 0);
+  }
+  if (tid == n_local - 1) {
+    offsets[n_local] = rows;
+    meta[0] = rows;
     meta[1] = nt;
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < n_local; i += blockDim.x) { counts[i] = cnt[i]; offsets[i] = off[i]; }
-  if (threadIdx.x == 0) offsets[n_local] = off[n_local];
   // Slot assignment.  Tokens are visited in index order by consecutive threads, so slots inside an expert are only
   // approximately token-ordered; every row is processed independently, so values do not depend on the order.
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    const int e = ids[i] - e0;
-    if (e >= 0 && e < n_local) {
-      const int s = off[e] + atomicAdd(&cur[e], 1);
-      slot_token[s] = i / k;
-      inv[i] = s;
-    } else {
-      inv[i] = -1;
-    }
+  for (int i = tid * 4; i < pairs; i += blockDim.x * 4) {
+    int e[4], s[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) e[j] = i + j < pairs ? ids[i + j] - e0 : -1;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) s[j] = e[j] >= 0 && e[j] < n_local ? atomicAdd(&cur[e[j]], 1) : -1;
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (i + j < pairs) {
+        if (s[j] >= 0) slot_token[s[j]] = (i + j) / k;
+        inv[i + j] = s[j];
+      }
   }
 }
 
@@ -192,7 +220,7 @@ extern "C" int b200_router_topk(const float* logits, long long ld, int M, int E,
 extern "C" int b200_moe_align(const int* ids, int M, int k, int e0, int n_local, int* counts, int* offsets, int* slot_token,
                               int* inv, void* tiles, int* meta, cudaStream_t stream) {
   if (M <= 0 || n_local <= 0 || n_local > 1024) return -1;
-  const size_t smem = static_cast<size_t>(3 * n_local + 1) * sizeof(int);
+  const size_t smem = static_cast<size_t>(2 * n_local) * sizeof(int);
   launch_ex(moe_align_kernel, dim3(1), dim3(1024), smem, stream, 0, ids, M, k, e0, n_local, counts, offsets, slot_token, inv,
                                               static_cast<int4*>(tiles), meta);
   cudaError_t e = cudaGetLastError();
