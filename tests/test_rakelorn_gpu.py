@@ -47,7 +47,7 @@ def i32(v):
 # ---------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("M,H,n,k,xg,yg", [(1, 3, 40, 24, 32, 40), (5, 1, 136, 64, 64, 136), (17, 6, 200, 77, 104, 208), (33, 4, 20, 130, 136, 24),
-                                            (64, 2, 300, 64, 96, 304), (65, 5, 64, 512, 512, 64), (200, 3, 130, 100, 104, 136)])
+                                            (64, 2, 300, 64, 96, 304), (65, 5, 64, 512, 512, 64), (200, 3, 130, 100, 104, 136), (8230, 2, 40, 24, 24, 40)])
 def test_linear_per_head_with_gate(M, H, n, k, xg, yg, dtype):
     from mojo_linuxperiments_b200.ops import dense as D
     g = gen(M)
